@@ -13,7 +13,8 @@
 //
 // Further options of ``attend`` (``AttnExtra``): ``chunk`` > 0 lets a query see only the keys of its own block of
 // ``chunk`` positions (blocks counted from position 0 of the sequence); ``gate`` multiplies head h's output row by
-// sigmoid(gate[t * gate_ld + h]) (float32 logits); ``out_scale`` multiplies it by a constant; ``out_stride`` is the
+// sigmoid(gate[t * gate_ld + h]) (float32 logits) or, with ``gate_elem``, element i of it by
+// sigmoid(gate[t * gate_ld + h * vd + i]); ``out_scale`` multiplies it by a constant; ``out_stride`` is the
 // distance between output rows, so that the heads may land in a column range of a wider tensor.
 //
 // A page of the cache holds the keys [G, page_size, d] and then the values [G, page_size, vd].
@@ -28,6 +29,7 @@ struct AttnExtra {
   int chunk;              // 0: none
   const float* gate;      // float32 logits, row t at t * gate_ld, head h at + h; null: none
   long long gate_ld;
+  int gate_elem;          // 1: one logit per output element (h * vd + i), 0: one per head
   float out_scale;
   long long out_stride;   // elements between output rows
 };
@@ -41,8 +43,12 @@ __device__ __forceinline__ int as_key_lo(int pos, int window, int chunk) {
 // What the finished row of (token t, head h) is multiplied by.
 __device__ __forceinline__ float as_out_factor(const AttnExtra& ex, int t, int h) {
   float f = ex.out_scale;
-  if (ex.gate) f *= 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.gate_ld + h]));
+  if (ex.gate && !ex.gate_elem) f *= 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.gate_ld + h]));
   return f;
+}
+// ... and element i of it once more.
+__device__ __forceinline__ float as_elem_gate(const AttnExtra& ex, int t, int h, int vd, int i) {
+  return ex.gate_elem ? 1.0f / (1.0f + expf(-ex.gate[(size_t)t * ex.gate_ld + (size_t)h * vd + i])) : 1.0f;
 }
 
 __device__ __forceinline__ float as_ld(const void* p, int code, size_t i) {
@@ -234,7 +240,7 @@ sink_attention_generic_kernel(const T* __restrict__ q, long long q_stride, T* __
 #pragma unroll
   for (int i = 0; i < AS_MAX_D / 32; i++) {
     const int idx = lane + 32 * i;
-    if (idx < vd) orow[idx] = from_float<T>(o[i] * inv);
+    if (idx < vd) orow[idx] = from_float<T>(o[i] * inv * as_elem_gate(ex, t, h, vd, idx));
   }
 }
 
@@ -244,15 +250,15 @@ extern "C" int qd_sink_attention_generic(const void* q, long long q_stride, void
                                          const void* kv, int dtype, const int* block_table, int max_blocks,
                                          const int* token_req, const int* positions, int n_tokens, int H, int G, int d,
                                          int vd, int page_size, float scale, int window, const float* sinks,
-                                         int chunk, const float* gate, long long gate_ld, float out_scale,
-                                         cudaStream_t stream) {
+                                         int chunk, const float* gate, long long gate_ld, int gate_elem,
+                                         float out_scale, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (d <= 0 || d > AS_MAX_D || vd <= 0 || vd > AS_MAX_D || G <= 0 || H % G != 0 || page_size <= 0)
     return QD_ERR_UNSUPPORTED;
   const long long items = (long long)n_tokens * H;
   const unsigned blocks = (unsigned)((items + AS_WARPS - 1) / AS_WARPS);
   const size_t smem = (size_t)AS_WARPS * d * sizeof(float);
-  const AttnExtra ex = {chunk, gate, gate_ld, out_scale, out_stride};
+  const AttnExtra ex = {chunk, gate, gate_ld, gate && gate_elem, out_scale, out_stride};
   if (dtype == QD_F32)
     qd_launch(sink_attention_generic_kernel<float>, dim3(blocks), dim3(AS_WARPS * 32), smem, stream, (const float*)q,
               q_stride, (float*)out, out_stride, (const float*)kv, block_table, max_blocks, token_req, positions,
@@ -495,7 +501,8 @@ sink_attention_mma_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, co
       const int col = n * 8 + 2 * tq;
       if (col < vd)
         *reinterpret_cast<unsigned*>(out + (size_t)t * ex.out_stride + (size_t)h * vd + col) =
-            ts_pack(o[n][2 * half] * f, o[n][2 * half + 1] * f);
+            ts_pack(o[n][2 * half] * f * as_elem_gate(ex, t, h, vd, col),
+                    o[n][2 * half + 1] * f * as_elem_gate(ex, t, h, vd, col + 1));
     }
   }
   if (splits == 1 || tickets == nullptr) return;            // without tickets a combine kernel follows
@@ -558,7 +565,8 @@ sink_attention_mma_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, co
       ay = fmaf(v.y, w, ay);
     }
     const float f = inv_l[row];
-    *reinterpret_cast<unsigned*>(out + (size_t)(t0 + tk_) * ex.out_stride + (size_t)h * vd + i) = ts_pack(ax * f, ay * f);
+    *reinterpret_cast<unsigned*>(out + (size_t)(t0 + tk_) * ex.out_stride + (size_t)h * vd + i) =
+        ts_pack(ax * f * as_elem_gate(ex, t0 + tk_, h, vd, i), ay * f * as_elem_gate(ex, t0 + tk_, h, vd, i + 1));
   }
 }
 
@@ -591,7 +599,8 @@ sink_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ 
       const float w = __shfl_sync(0xffffffffu, s < 32 ? wa : wb, s & 31);
       if (i < vd) acc = fmaf(po[(size_t)s * vd + i], w, acc);
     }
-    if (i < vd) out[(size_t)t_ * ex.out_stride + (size_t)h_ * vd + i] = __float2bfloat16_rn(acc * inv);
+    if (i < vd)
+      out[(size_t)t_ * ex.out_stride + (size_t)h_ * vd + i] = __float2bfloat16_rn(acc * inv * as_elem_gate(ex, t_, h_, vd, i));
   }
 }
 
@@ -605,13 +614,13 @@ extern "C" int qd_sink_attention_mma(const void* q, void* out, const void* kv, c
                                      int H, int G, int d, int vd, int page_size, float scale, int window,
                                      const float* sinks, int splits, float* part_o, float* part_ml,
                                      unsigned* tickets, int chunk, const float* gate, long long gate_ld,
-                                     float out_scale, long long out_stride, cudaStream_t stream) {
+                                     int gate_elem, float out_scale, long long out_stride, cudaStream_t stream) {
   if (n_tokens <= 0 || n_requests <= 0) return 0;
   if (G <= 0 || H % G || H / G > TS_ROWS || d <= 0 || vd <= 0 || d > 128 || vd > 128 || d % 8 || vd % 8 ||
       page_size <= 0 || splits < 1 || splits > 64 || G > 65535 || (splits > 1 && (!part_o || !part_ml)) ||
       out_stride < (long long)H * vd || (out_stride & 1))
     return QD_ERR_UNSUPPORTED;
-  const AttnExtra ex = {chunk, gate, gate_ld, out_scale, out_stride};
+  const AttnExtra ex = {chunk, gate, gate_ld, gate && gate_elem, out_scale, out_stride};
   const float scale_log2 = scale * 1.4426950408889634f;
   int page_shift = -1;
   if ((page_size & (page_size - 1)) == 0)

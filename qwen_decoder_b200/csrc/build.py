@@ -51,6 +51,8 @@ LIBRARIES: Dict[str, str] = {
     "attention_diff": "attention_diff.cu",
     "qkv_prep": "qkv_prep.cu",
     "time_mix": "time_mix.cu",
+    "linear_scan": "linear_scan.cu",
+    "group_norm": "group_norm.cu",
 }
 HEADERS = ["common.cuh", "entry_points.h"]
 # further files a library's source includes (hashed into its key)
@@ -59,6 +61,7 @@ EXTRA_DEPS: Dict[str, List[str]] = {
     "gated_block": ["short_conv.cuh"],
     "attention_diff": ["short_conv.cuh", "mma_sync.cuh"],
     "qkv_prep": ["short_conv.cuh"],
+    "linear_scan": ["short_conv.cuh"],
     "attention_sink": ["mma_sync.cuh"],
 }
 

@@ -596,8 +596,8 @@ __global__ void swiglu_vec_kernel(const bf16* __restrict__ gate_up, bf16* __rest
 // The same from the float32 partial sums of a split-K product: part [n_parts, T, 2F]; the shares are added
 // first, exactly (float32), and the result is rounded to bfloat16 once.  Four features per thread with 16-byte
 // loads, all shares of a thread's gate and up values asked for before any is used (in groups of four shares).
-__global__ void swiglu_partial_kernel(const float* __restrict__ part, int n_parts, bf16* __restrict__ out, int F4,
-                                      size_t n4, size_t part_stride4) {
+__global__ void swiglu_partial_kernel(const float* __restrict__ part, int n_parts, const float* __restrict__ bias,
+                                      bf16* __restrict__ out, int F4, size_t n4, size_t part_stride4) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -606,6 +606,7 @@ __global__ void swiglu_partial_kernel(const float* __restrict__ part, int n_part
   const int a = (int)(i - t * F4);
   const float4* base = reinterpret_cast<const float4*>(part) + t * 2 * F4 + a;
   float4 g = make_float4(0.f, 0.f, 0.f, 0.f), u = g;
+  if (bias) { g = reinterpret_cast<const float4*>(bias)[a]; u = reinterpret_cast<const float4*>(bias)[F4 + a]; }
   for (int p0 = 0; p0 < n_parts; p0 += 4) {
     float4 gv[4], uv[4];
 #pragma unroll
@@ -628,12 +629,15 @@ __global__ void swiglu_partial_kernel(const float* __restrict__ part, int n_part
   reinterpret_cast<uint2*>(out)[i] = o;
 }
 
-// out [T, F] bfloat16 = silu(sum_p part[p, t, f]) * (sum_p part[p, t, F + f]); F a multiple of 4, 16-byte aligned.
-extern "C" int qd_swiglu_partial(const float* part, int n_parts, void* out, int T, int F, cudaStream_t stream) {
+// out [T, F] bfloat16 = silu(bias[f] + sum_p part[p, t, f]) * (bias[F + f] + sum_p part[p, t, F + f]); bias [2F] or null;
+// F a multiple of 4, 16-byte aligned.
+extern "C" int qd_swiglu_partial(const float* part, int n_parts, const float* bias, void* out, int T, int F,
+                                 cudaStream_t stream) {
   if (T <= 0 || F <= 0) return 0;
-  if (n_parts < 1 || F % 4 != 0 || (((uintptr_t)part) & 15) || (((uintptr_t)out) & 7)) return QD_ERR_UNSUPPORTED;
+  if (n_parts < 1 || F % 4 != 0 || (((uintptr_t)part | (uintptr_t)bias) & 15) || (((uintptr_t)out) & 7))
+    return QD_ERR_UNSUPPORTED;
   const size_t n4 = (size_t)T * F / 4;
-  qd_launch(swiglu_partial_kernel, dim3((unsigned)((n4 + 127) / 128)), dim3(128), 0, stream, part, n_parts, (bf16*)out,
+  qd_launch(swiglu_partial_kernel, dim3((unsigned)((n4 + 127) / 128)), dim3(128), 0, stream, part, n_parts, bias, (bf16*)out,
             F / 4, n4, (size_t)T * 2 * F / 4);
   return qd_last_error();
 }

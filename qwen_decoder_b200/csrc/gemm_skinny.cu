@@ -134,6 +134,7 @@ gemm_skinny_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, long 
       float gate = 0.f, up = 0.f;
 #pragma unroll
       for (int w = 0; w < SK_WARPS; w++) { gate += red[w][row][tok]; up += red[w][row + 8][tok]; }
+      if (bias) { gate += bias[f]; up += bias[F + f]; }
       out[(size_t)tok * ldo + f] = from_float<TO>(gate / (1.0f + expf(-gate)) * up);
     }
   } else {
@@ -162,7 +163,7 @@ static int launch_skinny(const bf16* W, const bf16* X, long long ldx, const floa
   if (epi == EPI_SWIGLU) {
     dim3 grid((N / 2 + 7) / 8, 1);
     if (out_dtype != QD_BF16) return QD_ERR_UNSUPPORTED;
-    qd_launch(gemm_skinny_kernel<TN, EPI_SWIGLU, bf16>, dim3(grid), dim3(block), 0, stream, W, X, ldx, nullptr, (bf16*)out, ldo,
+    qd_launch(gemm_skinny_kernel<TN, EPI_SWIGLU, bf16>, dim3(grid), dim3(block), 0, stream, W, X, ldx, bias, (bf16*)out, ldo,
                                                                          nullptr, T, N, K, 1);
   } else if (epi == EPI_PARTIAL) {
     dim3 grid((N + 15) / 16, splits);
@@ -184,7 +185,7 @@ static int launch_skinny(const bf16* W, const bf16* X, long long ldx, const floa
 
 // epi 0: out[T, N] = X W^T + bias (out_dtype bf16 or f32).  epi 1: part[splits, T, N] float32 partial
 // sums over ``splits`` shares of K (no bias).  epi 2: W is [2F, K] = gate rows then up rows, N = 2F,
-// out[T, F] = silu(X Wg^T) * (X Wu^T), bfloat16.  X rows are ldx elements apart, out rows ldo.
+// out[T, F] = silu(X Wg^T + bias_g) * (X Wu^T + bias_u), bfloat16 (bias [2F] or null).  X rows are ldx elements apart, out rows ldo.
 extern "C" int qd_gemm_skinny(const void* W, const void* X, long long ldx, const float* bias, void* out,
                               int out_dtype, long long ldo, float* part, int T, int N, int K, int splits,
                               int epi, cudaStream_t stream) {

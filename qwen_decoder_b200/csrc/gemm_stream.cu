@@ -10,7 +10,7 @@
 // a stage (each a quarter of its k range) with 16-byte shared loads and feed mma.sync
 // m16n8k16 with the tokens as the N dimension; the 16-byte operand trick is the one of
 // gemm_skinny.cu.  After an item's last stage the four partial sums are added in shared
-// memory and the epilogue runs: store (+ bias), split-K partial sums, or SwiGLU.
+// memory and the epilogue runs: store (+ bias), split-K partial sums, or SwiGLU (+ bias on gate and up).
 // The producer starts before the programmatic-dependency wait (weights are written by no
 // kernel of the step); the consumers wait before they read the tokens.
 //
@@ -244,6 +244,7 @@ gemm_stream_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, long 
           gate += red[((size_t)w * 16 + row) * RED_LD + tok];
           up += red[((size_t)w * 16 + row + 8) * RED_LD + tok];
         }
+        if (bias) { gate += bias[f]; up += bias[F + f]; }
         out[(size_t)tok * ldo + f] = from_float<TO>(gate / (1.0f + expf(-gate)) * up);
       }
     } else {
@@ -472,6 +473,7 @@ gemm_stream_xres_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, 
           gate += red[((size_t)w * 16 + row) * RED_LD + tok];
           up += red[((size_t)w * 16 + row + 8) * RED_LD + tok];
         }
+        if (bias) { gate += bias[f]; up += bias[F + f]; }
         out[(size_t)tok * ldo + f] = from_float<TO>(gate / (1.0f + expf(-gate)) * up);
       }
     } else {
@@ -505,6 +507,7 @@ gemm_stream_xres_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, 
 #define FFN_SYNC_WORDS 64
 struct FfnArgs {
   const bf16* w1; const bf16* x1; long long ldx1; int N1, K1, n_tiles1;        // [2F, D], tokens [T, D]
+  const float* b1;                                                              // [2F] added before SwiGLU, or null
   bf16* h; long long ldh;                                                       // [T, F]
   const bf16* w2; int N2, K2, n_tiles2, splits2; float* part;                   // [D, F] -> [splits2, T, D]
   int T;
@@ -709,6 +712,7 @@ ffn_stream_kernel(const FfnArgs a) {
         gate += red[((size_t)w * 16 + row) * RED_LD + tok];
         up += red[((size_t)w * 16 + row + 8) * RED_LD + tok];
       }
+      if (a.b1) { gate += a.b1[f]; up += a.b1[F + f]; }
       a.h[(size_t)tok * a.ldh + f] = __float2bfloat16_rn(gate / (1.0f + expf(-gate)) * up);
     }
     asm volatile("bar.sync 1, %0;" ::"n"(ST_CONSUMERS * 32) : "memory");
@@ -863,11 +867,11 @@ extern "C" int qd_gemm_stream(const void* W, const void* X, long long ldx, const
 }
 
 // The feed-forward of up to 8 tokens in one launch: h = silu(x Wg^T) * (x Wu^T) (w1 = [Wg; Wu], [2F, D]) and
-// part[s] = partial sums of h W2^T over `splits2` shares of F.  `gbar`: 64 zeroed words of device memory that
+// part[s] = partial sums of h W2^T over `splits2` shares of F; `b1` [2F] (or null) is added to gate and up.  `gbar`: 64 zeroed words of device memory that
 // stay with the caller (the kernel leaves them zero for the next launch).  Refuses what it cannot take
 // (more than 8 tokens, D above 2,048, a share of F wider than 2,048, more CTAs than fit on the device at once).
-extern "C" int qd_ffn_stream(const void* w1, const void* x, long long ldx, void* h, long long ldh, const void* w2,
-                             float* part, int T, int D, int F, int splits2, unsigned* gbar, int max_ctas,
+extern "C" int qd_ffn_stream(const void* w1, const float* b1, const void* x, long long ldx, void* h, long long ldh,
+                             const void* w2, float* part, int T, int D, int F, int splits2, unsigned* gbar, int max_ctas,
                              long long* timeline, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (T > 8 || D <= 0 || F <= 0 || D % 8 != 0 || F % 8 != 0 || ldx % 8 != 0 || ldh % 8 != 0 || D > XR_KMAX ||
@@ -891,7 +895,7 @@ extern "C" int qd_ffn_stream(const void* w1, const void* x, long long ldx, void*
     return QD_ERR_UNSUPPORTED;
   }
   FfnArgs a;
-  a.w1 = (const bf16*)w1; a.x1 = (const bf16*)x; a.ldx1 = ldx; a.N1 = 2 * F; a.K1 = D; a.n_tiles1 = (F + 7) / 8;
+  a.w1 = (const bf16*)w1; a.b1 = b1; a.x1 = (const bf16*)x; a.ldx1 = ldx; a.N1 = 2 * F; a.K1 = D; a.n_tiles1 = (F + 7) / 8;
   a.h = (bf16*)h; a.ldh = ldh;
   a.w2 = (const bf16*)w2; a.N2 = D; a.K2 = F; a.n_tiles2 = (D + 15) / 16; a.splits2 = splits2; a.part = part;
   a.T = T; a.gbar = gbar; a.status = status; a.timeline = timeline;

@@ -268,7 +268,8 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
       tc_fence_after();
       const int feature = ft * TC_BM + lane_base + lane;           // within a half for SwiGLU
       const int n_feat = EPI == EPI_SWIGLU ? F : p.N;
-      const float bv = (EPI == EPI_STORE && bias && feature < n_feat) ? bias[feature] : 0.f;
+      const float bv = (EPI != EPI_PARTIAL && bias && feature < n_feat) ? bias[feature] : 0.f;
+      const float bu = (EPI == EPI_SWIGLU && bias && feature < n_feat) ? bias[F + feature] : 0.f;
       const unsigned t0 = tmem_base + ((unsigned)lane_base << 16) + buf * p.acc_cols;
       const int n_used = min(p.nacc, (kb1 - kb0) * (TC_BK / 16));    // accumulators this item wrote
       for (int c = 0; c < p.BN; c += 16) {
@@ -293,7 +294,8 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
             if (tok < p.T) {
               float a = v[i];
               if (EPI == EPI_SWIGLU) {
-                out[(size_t)tok * p.ldo + feature] = from_float<TO>(a / (1.0f + expf(-a)) * u[i]);
+                a += bv;
+                out[(size_t)tok * p.ldo + feature] = from_float<TO>(a / (1.0f + expf(-a)) * (u[i] + bu));
               } else if (EPI == EPI_PARTIAL) {
                 part[((size_t)sp * p.T + tok) * p.N + feature] = a;
               } else {

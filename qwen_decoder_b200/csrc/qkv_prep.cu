@@ -26,7 +26,7 @@ __device__ __forceinline__ void qp_st(void* p, int code, size_t i, float v) {
 }
 
 // The two elements of pair j of a head: (2j, 2j+1), or with half-split pairing (j, j + half) inside the rotated part
-// (pairs past it cover the elements from 2 half on, two by two).
+// (pairs past it cover the elements from 2 half on, two by two; an odd head size leaves the last pair's second out).
 __device__ __forceinline__ void qp_pair(int pairing, int half, int j, int& ia, int& ib) {
   if (pairing == 1 && j < half) { ia = j; ib = j + half; }
   else { ia = 2 * j; ib = 2 * j + 1; }
@@ -83,7 +83,7 @@ qkv_prep_kernel(QkvPrep a) {
   }
   const size_t page_elems = (size_t)G * a.page_size * (d + vd);
   const int pos = a.positions[t];
-  const int half = a.rotary_dim / 2, pairs = d / 2;
+  const int half = a.rotary_dim / 2, pairs = (d + 1) / 2;
   for (int s = warp; s < H + G; s += blockDim.x >> 5) {
     const bool is_q = s < H;
     if (!is_q && !a.write_kv) continue;
@@ -99,8 +99,9 @@ qkv_prep_kernel(QkvPrep a) {
       if (j >= pairs) continue;
       int ia, ib;
       qp_pair(a.pairing, half, j, ia, ib);
-      float xa = row[base + ia], yb = row[base + ib];
-      if (w) { xa *= f * w[ia]; yb *= f * w[ib]; }
+      const bool two = ib < d;
+      float xa = row[base + ia], yb = two ? row[base + ib] : 0.f;
+      if (w) { xa *= f * w[ia]; if (two) yb *= f * w[ib]; }
       if (a.norm_mode == 2 && !a.norm_after) ss = fmaf(xa, xa, fmaf(yb, yb, ss));
       x[i] = xa; y[i] = yb;
     }
@@ -133,7 +134,7 @@ qkv_prep_kernel(QkvPrep a) {
       int ia, ib;
       qp_pair(a.pairing, half, j, ia, ib);
       qp_st(out, oc, dst + ia, x[i] * fh);
-      qp_st(out, oc, dst + ib, y[i] * fh);
+      if (ib < d) qp_st(out, oc, dst + ib, y[i] * fh);
     }
   }
   if (!a.write_kv) return;
@@ -169,7 +170,7 @@ extern "C" int qd_qkv_prep(const float* u, long long ld, int T, int n_requests, 
                            cudaStream_t stream) {
   if (T <= 0) return 0;
   const long long C = (long long)H * d + (long long)G * d + (long long)G * vd;
-  if (d <= 0 || d > QP_MAX_D || (d & 1) || vd <= 0 || G <= 0 || H <= 0 || rotary_dim < 0 || rotary_dim > d ||
+  if (d <= 0 || d > QP_MAX_D || vd <= 0 || G <= 0 || H <= 0 || rotary_dim < 0 || rotary_dim > d ||
       (rotary_dim & 1) || taps < 0 || (taps > 1 && !state) || (taps > 0 && !conv_w) || norm_mode < 0 || norm_mode > 2 ||
       (norm_mode == 1 && (!wq || !wk)) || (rotary_dim > 0 && (!cos_t || !sin_t)) || n_requests > 65535)
     return QD_ERR_UNSUPPORTED;

@@ -219,14 +219,15 @@ def elementwise_plain_next() -> None:
     fn()
 
 
-def swiglu_partial(part: torch.Tensor, out: torch.Tensor) -> None:
+def swiglu_partial(part: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:
     """out[t, f] = silu(sum_p part[p, t, f]) * (sum_p part[p, t, F + f]) from the float32 partial sums
-    [n_parts, T, 2F] of a split-K gate/up product; out bfloat16."""
+    [n_parts, T, 2F] of a split-K gate/up product (plus ``bias`` float32 [2F], if given); out bfloat16."""
     T, F = out.shape
     assert part.dim() == 3 and tuple(part.shape[1:]) == (T, 2 * F) and part.dtype == torch.float32
     assert out.dtype == torch.bfloat16 and F % 4 == 0
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == 2 * F and bias.is_contiguous())
     _contig(part, "part"); _contig(out, "out")
-    _check(library("elementwise").qd_swiglu_partial(_ptr(part), _I(part.shape[0]), _ptr(out), _I(T), _I(F), _stream()),
+    _check(library("elementwise").qd_swiglu_partial(_ptr(part), _I(part.shape[0]), _ptr(bias), _ptr(out), _I(T), _I(F), _stream()),
            "swiglu_partial")
 
 
@@ -461,13 +462,16 @@ def gemm_skinny_partial(x: torch.Tensor, w: torch.Tensor, splits: int) -> torch.
     return part
 
 
-def gemm_skinny_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor) -> None:
-    """out[T, F] = silu(x @ Wg^T) * (x @ Wu^T) with w_gate_up = [Wg; Wu] of shape [2F, K]."""
+def gemm_skinny_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor,
+                       bias: Optional[torch.Tensor] = None) -> None:
+    """out[T, F] = silu(x @ Wg^T) * (x @ Wu^T) with w_gate_up = [Wg; Wu] of shape [2F, K]; ``bias`` float32 [2F]: added
+    to both products first."""
     T, K = x.shape
     N = w_gate_up.shape[0]
     assert skinny_supported(x, w_gate_up, 1 << 30) and out.shape == (T, N // 2) and out.dtype == torch.bfloat16
     _contig(w_gate_up, "w"); _contig(out, "out")
-    _skinny_call(x, w_gate_up, None, out, None, T, N, K, 1, EPI_SWIGLU, "gemm_skinny_swiglu")
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous())
+    _skinny_call(x, w_gate_up, bias, out, None, T, N, K, 1, EPI_SWIGLU, "gemm_skinny_swiglu")
 
 
 def ffn_stream_supported(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor) -> bool:
@@ -483,14 +487,16 @@ FFN_SYNC_WORDS = 64      # words of device memory a layer's one-launch feed-forw
 
 
 def ffn_stream(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, barrier: torch.Tensor,
-               timeline: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """float32 partial sums [splits, T, D] of (silu(x Wg^T) * (x Wu^T)) Wd^T for up to 8 tokens, in one
+               timeline: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """float32 partial sums [splits, T, D] of (silu(x Wg^T) * (x Wu^T)) Wd^T (``bias`` float32 [2F], if given, joins both
+    products of x) for up to 8 tokens, in one
     launch of the weight streamer: between the two products a CTA waits for the others' columns of h that its
     share of the second product reads, its producer warp meanwhile fetches the second product's first weights.  ``barrier``: ``FFN_SYNC_WORDS`` int32 words
     on the device, zero before their first use, that belong to the caller (no two launches that may run
     at the same time share them); every launch leaves them ready for the next.  ``timeline``: for measurements,
     int64 [CTAs, 8] that takes the kernel's own nanosecond stamps."""
     assert barrier.dtype == torch.int32 and barrier.numel() >= FFN_SYNC_WORDS and barrier.is_cuda
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == w_gate_up.shape[0] and bias.is_contiguous())
     T, D = x.shape
     F = w_down.shape[1]
     _contig(w_gate_up, "w_gate_up"); _contig(w_down, "w_down")
@@ -498,7 +504,7 @@ def ffn_stream(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, b
     h = torch.empty((T, F), dtype=torch.bfloat16, device=x.device)
     part = torch.empty((splits, T, D), dtype=torch.float32, device=x.device)
     _check(library("gemm_stream").qd_ffn_stream(
-        _ptr(w_gate_up), _ptr(x), _LL(x.stride(0)), _ptr(h), _LL(h.stride(0)), _ptr(w_down), _ptr(part), _I(T), _I(D),
+        _ptr(w_gate_up), _ptr(bias), _ptr(x), _LL(x.stride(0)), _ptr(h), _LL(h.stride(0)), _ptr(w_down), _ptr(part), _I(T), _I(D),
         _I(F), _I(splits), _ptr(barrier), _I(stream_max_ctas()), _ptr(timeline), _stream()), "ffn_stream")
     return part
 
@@ -1252,16 +1258,18 @@ def qk_norm_rope_write(qkv: torch.Tensor, H: int, G: int, d: int, vd: int, wq: O
 def sink_attention_generic(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, block_table: torch.Tensor,
                            token_req: torch.Tensor, positions: torch.Tensor, H: int, G: int, d: int, vd: int,
                            page_size: int, scale: float, window: int, sinks: Optional[torch.Tensor], chunk: int = 0,
-                           gate: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
+                           gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, gate_elem: bool = False) -> None:
     """Attention of every token over keys 0..pos (or the last ``window``; with ``chunk`` only those of the query's
     own block of ``chunk`` positions) of its request with a sink in the softmax's denominator (``sinks`` float32 [H],
     or None), values of size ``vd``; q [T, H*d], out [T, H*vd] (rows may be strided: a column range of a wider
     tensor); head h's output is multiplied by ``out_scale`` and, with ``gate`` (float32 [T, >= H] logits, rows may be
-    strided), by sigmoid(gate[t, h]); float32 arithmetic, any sizes."""
+    strided), by sigmoid(gate[t, h]) or, with ``gate_elem`` (gate [T, >= H*vd]), element by element by
+    sigmoid(gate[t, h*vd + i]); float32 arithmetic, any sizes."""
     T = q.shape[0]
     assert q.shape == (T, H * d) and out.shape == (T, H * vd) and q.dtype == out.dtype == kv.dtype
     assert q.stride(1) == 1 and out.stride(1) == 1
     assert gate is None or (gate.dtype == torch.float32 and gate.shape[0] == T and gate.stride(1) == 1)
+    assert gate is None or gate.shape[1] >= (H * vd if gate_elem else H)
     assert kv.numel() % (G * page_size * (d + vd)) == 0
     assert block_table.dtype == torch.int32 and block_table.dim() == 2
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == H)
@@ -1270,7 +1278,7 @@ def sink_attention_generic(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor,
         _ptr(q), _LL(q.stride(0)), _ptr(out), _LL(out.stride(0)), _ptr(kv), _I(dtype_code(q.dtype)), _ptr(block_table),
         _I(block_table.shape[1]), _ptr(token_req), _ptr(positions), _I(T), _I(H), _I(G), _I(d), _I(vd), _I(page_size),
         _F(scale), _I(window), _ptr(sinks), _I(chunk), _ptr(gate), _LL(gate.stride(0) if gate is not None else 0),
-        _F(out_scale), _stream()), "sink_attention_generic")
+        _I(1 if gate_elem else 0), _F(out_scale), _stream()), "sink_attention_generic")
 
 
 SINK_MMA_ROWS = 64       # rows, (token, head within the group) pairs, of one tile of the tensor-core kernel
@@ -1287,14 +1295,15 @@ def sink_attention_mma(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, blo
                        cu_tokens: torch.Tensor, start_pos: torch.Tensor, n_requests: int, n_tokens: int, H: int, G: int,
                        d: int, vd: int, page_size: int, scale: float, window: int, sinks: Optional[torch.Tensor],
                        splits: int = 1, chunk: int = 0, gate: Optional[torch.Tensor] = None,
-                       out_scale: float = 1.0) -> None:
+                       out_scale: float = 1.0, gate_elem: bool = False) -> None:
     """``sink_attention_generic`` on tensor cores for portions of ``n_requests`` requests (rows cu_tokens[r] ..
     cu_tokens[r+1]-1 of q and out, at positions start_pos[r]..): a decoded token is a portion of one.  ``splits`` > 1
     shares every tile's keys among that many CTAs (for steps of few tokens over long contexts).  ``chunk``, ``gate``,
-    ``out_scale`` and strided rows of ``out`` as for the generic kernel."""
+    ``gate_elem``, ``out_scale`` and strided rows of ``out`` as for the generic kernel."""
     assert q.dtype == out.dtype == kv.dtype == torch.bfloat16 and q.shape[1] == H * d and out.shape[1] == H * vd
     assert out.stride(1) == 1 and out.stride(0) % 2 == 0
     assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
+    assert gate is None or gate.shape[1] >= (H * vd if gate_elem else H)
     assert kv.numel() % (G * page_size * (d + vd)) == 0
     assert block_table.dtype == torch.int32 and block_table.dim() == 2 and block_table.shape[0] >= n_requests
     assert cu_tokens.dtype == torch.int32 and start_pos.dtype == torch.int32
@@ -1315,7 +1324,8 @@ def sink_attention_mma(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, blo
         _ptr(q), _ptr(out), _ptr(kv), _ptr(block_table), _I(block_table.shape[1]), _ptr(cu_tokens), _ptr(start_pos),
         _I(n_requests), _I(n_tokens), _I(tiles), _I(H), _I(G), _I(d), _I(vd), _I(page_size), _F(scale), _I(window),
         _ptr(sinks), _I(splits), _ptr(part_o), _ptr(part_ml), _ptr(tickets), _I(chunk), _ptr(gate),
-        _LL(gate.stride(0) if gate is not None else 0), _F(out_scale), _LL(out.stride(0)), _stream()),
+        _LL(gate.stride(0) if gate is not None else 0), _I(1 if gate_elem else 0), _F(out_scale), _LL(out.stride(0)),
+        _stream()),
         "sink_attention_mma")
     if splits > 1 and tickets is None:
         _launch_count[0] += 1
@@ -1422,6 +1432,121 @@ def tm_finish(o: torch.Tensor, g: torch.Tensor, norm: torch.Tensor, H: int, d: i
         _I(dtype_code(out.dtype)), _LL(out.stride(0)), _ptr(h), _I(dtype_code(h.dtype)), _I(h.shape[1]), _ptr(state),
         _LL(state.stride(0)), _LL(prev_off), _ptr(ctx.token_request), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots),
         _I(1 if write_state else 0), _stream()), "tm_finish")
+
+
+# ------------------------------------------------------------------ linear attention with one decay per head and token
+LINEAR_PADS = (16, 32, 48, 64, 96, 128, 256)      # what a head of queries and keys is padded to
+LINEAR_MAX_VDIM = 8192
+
+
+def linear_pad(d: int) -> int:
+    for p in LINEAR_PADS:
+        if d <= p:
+            return p
+    raise KernelError(f"linear attention: a query/key head of {d} exceeds {LINEAR_PADS[-1]}")
+
+
+def linear_prep(u: torch.Tensor, H: int, G: int, d: int, dv: int, conv_w: Optional[torch.Tensor],
+                state: Optional[torch.Tensor], conv_off: int, ctx, update_state: bool, unit_eps: Optional[float],
+                rotary_dim: int, pairing: int, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], q_scale: float,
+                k_scale: float, b_off: int, a_off: int, A_log: Optional[torch.Tensor], dt_bias: Optional[torch.Tensor]):
+    """From the float32 sums u [T, >= 2*G*d + H*dv] (q | k | v | ...; rows may be strided): (q, k, v, beta, g) for
+    ``linear_scan``.  With ``conv_w`` (float32 [2*G*d + H*dv, taps]) every channel of q, k and v passes a causal
+    convolution (the last taps - 1 inputs of a request live at ``conv_off`` of its row of ``state`` and are moved on
+    when ``update_state``) and silu; else v is a view of u.  ``unit_eps``: q and k of every head divided by
+    sqrt(sum of squares + unit_eps).  The first ``rotary_dim`` elements of a head turn by the table rows of
+    ``ctx.positions``; then q times ``q_scale``, k times ``k_scale``.  ``b_off`` / ``a_off`` >= 0: the columns of u whose
+    sigmoid is beta, and g = exp(-exp(A_log) softplus(u + dt_bias)); None otherwise."""
+    T = u.shape[0]
+    C = 2 * G * d + H * dv
+    assert u.dtype == torch.float32 and u.stride(1) == 1 and u.shape[1] >= max(C, b_off + H, a_off + H)
+    taps = 0
+    if conv_w is not None:
+        taps = conv_w.shape[1]
+        assert conv_w.shape == (C, taps) and conv_w.dtype == torch.float32 and conv_w.is_contiguous()
+        assert taps == 1 or (state is not None and state.dtype == torch.float32 and state.is_contiguous())
+    if rotary_dim:
+        assert cos.dtype == sin.dtype == torch.float32 and cos.shape[1] == rotary_dim // 2
+    if a_off >= 0:
+        assert A_log.dtype == dt_bias.dtype == torch.float32 and A_log.numel() == dt_bias.numel() == H
+    DP = linear_pad(d)
+    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=u.device)
+    q, k = new(T, G, DP), new(T, G, DP)
+    v = new(T, H * dv) if taps else u[:, 2 * G * d:C]
+    beta = new(T, H) if b_off >= 0 else None
+    g = new(T, H) if a_off >= 0 else None
+    _check(library("linear_scan").qd_linear_prep(
+        _ptr(u), _LL(u.stride(0)), _I(T), _I(ctx.num_requests), _I(H), _I(G), _I(d), _I(dv), _I(DP), _I(taps), _ptr(conv_w),
+        _ptr(state if taps > 1 else None), _LL(state.stride(0) if state is not None else 0), _LL(conv_off),
+        _ptr(ctx.token_request), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _I(1 if update_state else 0),
+        _I(0 if unit_eps is None else 1), _F(unit_eps or 0.0), _I(rotary_dim), _I(pairing), _ptr(cos), _ptr(sin),
+        _ptr(ctx.positions), _F(q_scale), _F(k_scale), _I(b_off), _I(a_off), _ptr(A_log), _ptr(dt_bias), _ptr(q), _ptr(k),
+        _ptr(v if taps else None), _ptr(beta), _ptr(g), _stream()), "linear_prep")
+    if update_state and taps > 1 and T != ctx.num_requests:
+        _launch_count[0] += 1
+    return q, k, v, beta, g
+
+
+def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: Optional[torch.Tensor], H: int,
+                d: int, dv: int, state: torch.Tensor, s_off: int, ctx, write_state: bool, gate: torch.Tensor,
+                norm: Optional[torch.Tensor], eps: float, out_scale: float, out: torch.Tensor) -> None:
+    """Per (request, head), token by token: S <- g S;  x = v, or with ``beta`` (the delta rule) beta (v - S^T k);
+    S <- S + k x^T;  o = S^T q;  out[t, head] = o / sqrt(mean(o^2) + eps) * norm * silu(gate) * out_scale.  q, k float32
+    [T, G, linear_pad(d)], v float32 [T, H*dv] (rows may be strided), g float32 [T, H] or [H] (the same for every token),
+    gate float32 [T, H*dv] logits (rows may be strided), norm float32 [dv] or None; S [H, dv, d] float32 at ``s_off`` of
+    the request's row of ``state``; out [T, H*dv] (rows may be strided)."""
+    T, G, DP = q.shape
+    assert q.dtype == k.dtype == v.dtype == g.dtype == gate.dtype == torch.float32 and k.shape == q.shape
+    assert v.shape == gate.shape == out.shape == (T, H * dv) and v.stride(1) == gate.stride(1) == out.stride(1) == 1
+    assert g.shape in ((T, H), (H,)) and (beta is None or (beta.shape == (T, H) and beta.dtype == torch.float32))
+    assert norm is None or (norm.dtype == torch.float32 and norm.numel() == dv)
+    assert state.dtype == torch.float32 and s_off + H * dv * d <= state.shape[1]
+    for n, t in (("q", q), ("k", k), ("g", g), ("state", state)):
+        _contig(t, n)
+    single = T == ctx.num_requests
+    o = None if single else torch.empty((T, H * dv), dtype=torch.float32, device=q.device)
+    _check(library("linear_scan").qd_linear_scan(
+        _ptr(q), _ptr(k), _ptr(v), _LL(v.stride(0)), _ptr(g), _I(H if g.dim() == 2 else 0), _ptr(beta), _I(T),
+        _I(ctx.num_requests), _I(H), _I(G), _I(d), _I(dv), _I(DP), _ptr(state), _LL(state.stride(0)), _LL(s_off),
+        _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _I(1 if write_state else 0), _ptr(o), _ptr(gate), _LL(gate.stride(0)),
+        _ptr(norm), _F(eps), _F(out_scale), _ptr(out), _I(dtype_code(out.dtype)), _LL(out.stride(0)), _stream()),
+        "linear_scan")
+    if not single:
+        _launch_count[0] += 1
+
+
+# ------------------------------------------------------------------ norms in groups, before and after a branch
+def group_add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], post=None, delta_bias: Optional[torch.Tensor] = None,
+                   weight: Optional[torch.Tensor] = None, eps: float = 0.0, groups: int = 1,
+                   out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+                   write_back: bool = True) -> None:
+    """x += y, y = delta (+ ``delta_bias`` [D]; delta [T, D], or float32 partial sums [n, T, D] that are added up), or with
+    ``post`` = (w, eps, groups) x += G(y; w, eps, groups); with ``weight`` also out[r] = G(x[s]; weight, eps, groups),
+    s = rows[r] (or r).  G cuts a row into ``groups`` equal parts, divides each by its own sqrt(mean(part^2) + eps) and
+    multiplies the whole by the weight.  ``write_back`` False leaves x as it was (the norm still sees the sum)."""
+    T, D = x.shape
+    assert x.dtype == torch.float32
+    _contig(x, "x")
+    n_parts = 1
+    if delta is not None:
+        if delta.dim() == 3:
+            n_parts = delta.shape[0]
+            assert delta.dtype == torch.float32
+        assert tuple(delta.shape[-2:]) == (T, D)
+        _contig(delta, "delta")
+    pw, pe, pg = post if post is not None else (None, 0.0, 1)
+    f32 = lambda t: t is None or (t.dtype == torch.float32 and t.numel() == D and t.is_contiguous())
+    assert f32(pw) and f32(delta_bias) and f32(weight)
+    n_rows = T
+    if weight is not None:
+        n_rows = out.shape[0]
+        assert out.shape == (n_rows, D) and (rows is None or (rows.dtype == torch.int32 and rows.numel() == n_rows))
+        _contig(out, "out")
+    _check(library("group_norm").qd_group_add_norm(
+        _ptr(x), _ptr(delta), _I(dtype_code(delta.dtype) if delta is not None else 0), _I(n_parts), _LL(T * D),
+        _ptr(delta_bias), _ptr(pw), _F(pe), _I(pg), _ptr(weight), _F(eps), _I(groups), _ptr(out),
+        _I(dtype_code(out.dtype) if out is not None else 0), _ptr(rows), _I(n_rows), _I(D), _I(1 if write_back else 0),
+        _stream()), "group_add_norm")
 
 
 # ------------------------------------------------------------------ the layers of a prompt step from native code

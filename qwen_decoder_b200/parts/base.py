@@ -50,7 +50,8 @@ class ResidualStream:
     """The residual sum of a step: ``x`` float32 [T, D], and a branch output ``delta`` that has
     not been added yet (the next norm's kernel adds it).  Blocks whose two branches read the same
     x leave a second output pending too (``delta2``), and a pending output may be one that joins
-    unit-normalised: ``delta_unit`` = (u float32 [D], eps) means x += delta / sqrt(mean(delta^2) + eps) * u.
+    unit-normalised: ``delta_unit`` = (u float32 [D], eps) means x += delta / sqrt(mean(delta^2) + eps) * u; or it joins
+    through a norm in groups of its own (``delta_post``), after a bias that its product left out (``delta_bias``).
     A norm that takes only the plain form calls ``settle()`` first."""
 
     def __init__(self, x: torch.Tensor):
@@ -62,15 +63,23 @@ class ResidualStream:
         self.delta_gate: Optional[torch.Tensor] = None      # float32 logits [T, D]: the pending branch joins times their sigmoid
         self.delta_gate_bias: Optional[torch.Tensor] = None  # float32 [D]: added to every row of the logits first
         self.delta_mult = 1.0                               # a constant on what is pending (both outputs of a pair)
+        self.delta_post = None                              # (w, eps, groups): the pending branch joins as its grouped norm
+        self.delta_bias: Optional[torch.Tensor] = None      # float32 [D]: added to the pending branch before that norm
         self.origin: Optional[torch.Tensor] = None          # the embedding output, kept when a block reads it again
 
     def push(self, delta: torch.Tensor, scale: Optional[torch.Tensor] = None, unit=None,
-             gate: Optional[torch.Tensor] = None, gate_bias: Optional[torch.Tensor] = None, mult: float = 1.0) -> None:
+             gate: Optional[torch.Tensor] = None, gate_bias: Optional[torch.Tensor] = None, mult: float = 1.0,
+             post=None, bias: Optional[torch.Tensor] = None) -> None:
         """Hand over a branch output (times ``scale`` along D, or times sigmoid(``gate`` + ``gate_bias``) element by
-        element, if given; times the constant ``mult``); what is still pending is added first."""
+        element, if given; times the constant ``mult``; or with ``bias`` added and then through the grouped norm
+        ``post`` = (w, eps, groups)); what is still pending is added first."""
         self.flush()
         if mult != 1.0 and (scale is not None or gate is not None):
             raise ValueError("a constant on a branch that has a layer scale or a gate is not supported")
+        if (post is not None or bias is not None) and \
+                (mult != 1.0 or scale is not None or gate is not None or unit is not None):
+            raise ValueError("a branch with a norm or a bias of its own takes no constant, layer scale, gate or unit norm")
+        self.delta_post, self.delta_bias = post, bias
         self.delta_mult = float(mult)
         self.delta = delta
         self.delta_scale = scale
@@ -94,20 +103,24 @@ class ResidualStream:
 
     def clear(self) -> None:
         self.delta = self.delta_scale = self.delta_unit = self.delta2 = self.delta_gate = None
-        self.delta_gate_bias = None
+        self.delta_gate_bias = self.delta_post = self.delta_bias = None
         self.delta_mult = 1.0
 
-    def settle(self, gated_ok: bool = False) -> None:
+    def settle(self, gated_ok: bool = False, post_ok: bool = False) -> None:
         """Add what only ``flush`` can add (a second output, a unit-normalised one, and -- unless the caller's own
-        kernel takes it, ``gated_ok`` -- a gated one); a plain pending delta stays."""
+        kernel takes it, ``gated_ok`` / ``post_ok`` -- a gated one or one with a norm or bias of its own); a plain
+        pending delta stays."""
         if self.delta2 is not None or self.delta_unit is not None or self.delta_mult != 1.0 or \
-                (self.delta_gate is not None and not gated_ok):
+                (self.delta_gate is not None and not gated_ok) or \
+                ((self.delta_post is not None or self.delta_bias is not None) and not post_ok):
             self.flush()
 
     def flush(self) -> None:
         if self.delta is None and self.delta2 is None:
             return
-        if self.delta_gate is not None:
+        if self.delta_post is not None or self.delta_bias is not None:
+            kernels.group_add_norm(self.x, self.delta, self.delta_post, self.delta_bias)
+        elif self.delta_gate is not None:
             if self.delta2 is not None or self.delta_unit is not None or self.delta_scale is not None:
                 raise ValueError("a gated branch beside a second, a scaled or a unit-normalised one is not supported")
             kernels.gated_add_norm(self.x, self.delta, self.delta_gate, gate_bias=self.delta_gate_bias)

@@ -180,7 +180,8 @@ class ParallelSideBlock(Block):
         T, dev = stream.x.shape[0], stream.x.device
         n1, n2 = self.norm1, self.norm2
         if type(n1) in (TanhNorm, RMSNorm) and (n2 is None or type(n2) in (TanhNorm, RMSNorm)) and \
-                stream.delta_scale is None and stream.delta_gate is None:
+                stream.delta_scale is None and stream.delta_gate is None and stream.delta_post is None and \
+                stream.delta_bias is None:
             h1 = torch.empty((T, self.size), dtype=self.dtype, device=dev)
             h2 = torch.empty((T, self.size), dtype=self.dtype, device=dev) if n2 is not None else None
             kernels.add_tanh_norm(stream.x, stream.pending(),
@@ -303,6 +304,52 @@ class GatedPreNormBlock(Block):
             h = self.norm2.forward(stream, self.dtype)
             g = self._gate_logits(self.gate2, h)
             stream.push(self.feed_forward.forward(h, ctx), gate=g, gate_bias=self.gate2.bias)
+
+
+@register_part("block", "pre_post_norm")
+class PrePostNormBlock(Block):
+    """A norm before and a norm after each branch:
+
+        x += norm_out1(mixer(norm_in1(x)));   x += norm_out2(feed_forward(norm_in2(x)))   (a layer may have no feed-forward)
+
+    A branch's output waits on the stream with its norm (and the bias its last product left out); the next norm's kernel
+    norms it, adds it and norms the sum, one launch between two branches."""
+    norm_roles = ("input", "mixer_out", "post_mixer", "feed_forward_out")
+
+    def __init__(self, mixer: Mixer, feed_forward, norms: Dict[str, Norm]):
+        need = self.norm_roles if feed_forward is not None else self.norm_roles[:2]
+        missing = [r for r in need if r not in norms]
+        if missing:
+            raise ValueError(f"pre_post_norm block needs norms {need}, missing {missing}")
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.norms = [norms[r] for r in need]
+        for n in self.norms[1::2]:
+            if not hasattr(n, "as_post"):
+                raise ValueError(f"pre_post_norm block: {type(n).__name__} cannot norm a branch's output")
+
+    def parts(self):
+        return self.norms + [p for p in (self.mixer, self.feed_forward) if p is not None]
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [s for p in self.parts() for s in p.tensor_specs()]
+
+    def bind(self, source: TensorSource, dtype: torch.dtype, device: torch.device) -> None:
+        self.dtype = dtype
+        for p in self.parts():
+            p.bind(source, dtype, device)
+
+    def forward(self, stream: ResidualStream, ctx, cache) -> None:
+        h = self.norms[0].forward(stream, self.dtype)
+        stream.push(self.mixer.forward(h, ctx, cache), post=self.norms[1].as_post())
+        if self.feed_forward is None:
+            return
+        h = self.norms[2].forward(stream, self.dtype)
+        ff, bias = self.feed_forward, None
+        if hasattr(ff, "forward_without_bias"):
+            delta, bias = ff.forward_without_bias(h, ctx)
+        else:
+            delta = ff.forward(h, ctx)
+        stream.push(delta, post=self.norms[3].as_post(), bias=bias)
 
 
 @register_part("block", "loop_input")

@@ -19,6 +19,15 @@ from ..weights.loader import TensorSource, TensorSpec
 from . import matmul_backend
 
 
+def pad_rows(weight: torch.Tensor, multiple: int) -> torch.Tensor:
+    """The matrix with zero rows appended up to a multiple of ``multiple`` (products of whole 16-byte rows of outputs run
+    on the faster kernels); nobody reads the outputs of those rows."""
+    extra = -weight.shape[0] % multiple
+    if not extra:
+        return weight.contiguous()
+    return torch.cat([weight, weight.new_zeros((extra, weight.shape[1]))], dim=0).contiguous()
+
+
 class Linear:
     def __init__(self, in_features: int, pieces: Sequence[Tuple[str, int]], bias: bool,
                  weight_suffix: str = ".weight", bias_suffix: str = ".bias"):
@@ -57,15 +66,20 @@ class Linear:
         matmul_backend.linear(x, self.weight, self.bias, out)
         return out
 
-    def forward_partial(self, x: torch.Tensor) -> torch.Tensor:
+    def forward_partial(self, x: torch.Tensor, with_bias: bool = True) -> torch.Tensor:
         """The product as something a residual stream can take: [T, N] in x's dtype, or -- from the
         few-token kernel -- float32 partial sums [n_parts, T, N] (bias not added) that the next
-        norm's kernel adds up."""
-        if self.bias is None and matmul_backend.use_skinny(x, self.weight):
+        norm's kernel adds up.  ``with_bias`` False leaves the bias to the caller."""
+        bias = self.bias if with_bias else None
+        if bias is None and matmul_backend.use_skinny(x, self.weight):
             matmul_backend.counters["own"] += 1
             return kernels.gemm_skinny_partial(x, self.weight, kernels.skinny_splits(self.out_features, self.in_features, x.shape[0]))
-        if self.bias is None and x.is_cuda and x.dtype == torch.bfloat16 and x.is_contiguous():
+        if bias is None and x.is_cuda and x.dtype == torch.bfloat16 and x.is_contiguous():
             shares = matmul_backend.library_shares(x.shape[0], self.out_features, self.in_features)
             if shares:
                 return matmul_backend.linear_partial_library(x, self.weight, shares)
+        if bias is not self.bias:
+            out = torch.empty((x.shape[0], self.out_features), dtype=x.dtype, device=x.device)
+            matmul_backend.linear(x, self.weight, None, out)
+            return out
         return self.forward(x)

@@ -24,6 +24,7 @@ from .linear import Linear
 from . import attention as _attention, block as _block, mlp as _mlp, norm as _norm, rotary as _rotary  # noqa: F401
 from . import latent_attention as _latent, mamba2 as _mamba2, moe as _moe, sink_attention as _sink  # noqa: F401
 from . import diff_attention as _diff, masked_attention as _masked, side_by_side as _side, time_mix as _tmix  # noqa: F401
+from . import linear_attention as _linear_attention  # noqa: F401
 
 
 class DecoderModel:

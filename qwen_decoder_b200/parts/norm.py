@@ -99,12 +99,50 @@ class TanhNorm(Norm):
 
     def forward(self, stream: ResidualStream, out_dtype: torch.dtype,
                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-        if stream.delta_scale is not None:
+        if stream.delta_scale is not None or stream.delta_post is not None or stream.delta_bias is not None:
             stream.flush()
         n = stream.x.shape[0] if rows is None else rows.numel()
         out = torch.empty((n, self.size), dtype=out_dtype, device=stream.x.device)
         kernels.add_tanh_norm(stream.x, stream.pending(), [self.launch_params(out)], rows=rows,
                               write_back=rows is None)
+        if rows is None:
+            stream.clear()
+        return out
+
+
+@register_part("norm", "group_rmsnorm")
+class GroupRMSNorm(Norm):
+    """RMS norm in groups: the row is cut into ``groups`` equal consecutive parts, each is divided by its own
+    sqrt(mean(part^2) + eps), and the whole is multiplied by w (float32 arithmetic).  The kernel first adds the branch
+    output that is pending on the stream, which may itself join through such a norm (``delta_post``): the norm after one
+    branch and the norm before the next are one launch (``csrc/group_norm.cu``)."""
+
+    def __init__(self, size: int, eps: float, groups: int = 1, prefix: str = "", tensor: str = "weight"):
+        if groups < 1 or size % groups:
+            raise ValueError(f"group_rmsnorm: groups ({groups}) must divide the size ({size})")
+        self.size, self.eps, self.groups = size, float(eps), int(groups)
+        self.prefix, self.tensor = prefix, tensor
+        self.weight: Optional[torch.Tensor] = None
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [TensorSpec(f"{self.prefix}{self.tensor}", (self.size,), init="around_one")]
+
+    def bind(self, source: TensorSource, dtype: torch.dtype, device: torch.device) -> None:
+        self.weight = source.get(f"{self.prefix}{self.tensor}").to(device=device, dtype=torch.float32).contiguous()
+
+    def as_post(self):
+        """This norm on a branch's output, as the residual stream takes it."""
+        return (self.weight, self.eps, self.groups)
+
+    def forward(self, stream: ResidualStream, out_dtype: torch.dtype,
+                rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if stream.delta_scale is not None:
+            stream.flush()
+        stream.settle(post_ok=True)
+        n = stream.x.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, self.size), dtype=out_dtype, device=stream.x.device)
+        kernels.group_add_norm(stream.x, stream.delta, stream.delta_post, stream.delta_bias, self.weight, self.eps,
+                               self.groups, out, rows=rows, write_back=rows is None)
         if rows is None:
             stream.clear()
         return out

@@ -16,6 +16,8 @@ theta_p / factor * r_p + theta_p * (1 - r_p), and every cosine and sine is multi
 wavelength l_p = 2 pi / theta_p, pair p keeps theta_p where l_p < original / high, turns at theta_p / factor where
 l_p > original / low, and between the two at (1 - s) theta_p / factor + s theta_p with
 s = (original / l_p - low) / (high - low); cosines and sines keep their size.
+
+``scaling`` with ``kind`` = "linear" (key factor) divides every rate by the factor.
 """
 from __future__ import annotations
 
@@ -52,8 +54,12 @@ class Rotary(PositionEncoding):
                 scaling = {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}
                 if scaling["factor"] <= 0 or scaling["original"] <= 0 or scaling["fast"] <= 0 or scaling["slow"] <= 0:
                     raise ValueError("rotary scaling: factor, original, fast and slow must be positive")
+            elif self.scaling_kind == "linear":
+                scaling = {"factor": float(scaling["factor"])}
+                if scaling["factor"] <= 0:
+                    raise ValueError("rotary scaling: factor must be positive")
             else:
-                raise ValueError(f"rotary scaling: kind must be 'ramp' or 'bands', got {self.scaling_kind!r}")
+                raise ValueError(f"rotary scaling: kind must be 'ramp', 'bands' or 'linear', got {self.scaling_kind!r}")
         self.scaling = scaling
         self.cos: Optional[torch.Tensor] = None
         self.sin: Optional[torch.Tensor] = None
@@ -70,6 +76,8 @@ class Rotary(PositionEncoding):
             between = (1.0 - blend) * inv_freq / sc["factor"] + blend * inv_freq
             inv_freq = torch.where(wavelength < sc["original"] / sc["high"], inv_freq,
                                    torch.where(wavelength > sc["original"] / sc["low"], inv_freq / sc["factor"], between))
+        elif self.scaling_kind == "linear":
+            inv_freq = inv_freq / self.scaling["factor"]
         elif self.scaling is not None:
             import math
             sc = self.scaling

@@ -8,6 +8,9 @@ sum_b scale_b Wo_b y_b = [Wo_1 | Wo_2 | ...] [scale_1 y_1 ; scale_2 y_2 ; ...], 
 into column ranges of ONE tensor and one product with the output matrices laid side by side finishes all of them.
 At most one branch may keep pages; the per-request states follow one another in one float32 state row.
 
+Where every branch begins with ONE stacked product of the same input (it has ``stacked`` and takes the product's sums as
+``u``), the branches' matrices are stacked too: one product serves all of them, and each reads its own columns.
+
 ``branches``: a list of {"name": registered mixer, "params": its parameters (``prefix`` relative to this mixer's),
 "scale": its weight}.
 """
@@ -21,7 +24,8 @@ from ..cache import FixedState
 from ..config.registry import create_part, register_part
 from ..weights.loader import TensorSource, TensorSpec
 from .base import Mixer, PagedCacheView, RunCacheView, StateCacheView
-from .linear import Linear
+from .linear import Linear, pad_rows
+from . import matmul_backend
 
 
 @register_part("mixer", "side_by_side")
@@ -71,6 +75,17 @@ class SideBySide(Mixer):
             m.bind(source, dtype, device)
         ws = [source.get(f"{m.out_stem}{self.sfx}").to(device=device, dtype=dtype) for m in self.mixers]
         self.out.bind_tensor(torch.cat(ws, dim=1).contiguous())
+        self.inp = None
+        if all(getattr(m, "stacked", None) is not None and m.stacked_bias is None for m in self.mixers):
+            rows = [m.stacked.shape[0] for m in self.mixers]
+            self.inp = pad_rows(torch.cat([m.stacked for m in self.mixers], dim=0), 8)
+            self.inp_rows, lo = [], 0
+            for m, n in zip(self.mixers, rows):          # the branches keep views: nothing is held twice
+                m.stacked = self.inp[lo:lo + n]
+                if hasattr(m, "release_inputs"):
+                    m.release_inputs()
+                self.inp_rows.append((lo, lo + n))
+                lo += n
 
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
         if isinstance(cache, RunCacheView):
@@ -80,10 +95,14 @@ class SideBySide(Mixer):
         else:
             paged, state, base, write = cache, None, 0, getattr(cache, "write", True)
         y = torch.empty((x.shape[0], sum(self.widths)), dtype=x.dtype, device=x.device)
-        lo = 0
-        for m, scale, off, width in zip(self.mixers, self.scales, self.offsets, self.widths):
+        lo, u = 0, None
+        if self.inp is not None:
+            u = torch.empty((x.shape[0], self.inp.shape[0]), dtype=torch.float32, device=x.device)
+            matmul_backend.linear(x, self.inp, None, u)
+        for i, (m, scale, off, width) in enumerate(zip(self.mixers, self.scales, self.offsets, self.widths)):
+            kw = {} if u is None else {"u": u[:, self.inp_rows[i][0]:self.inp_rows[i][1]]}
             view = RunCacheView(paged=paged if m.paged_need() is not None else None, state=state,
                                 state_off=base + off, write=write)
-            m.inner(x, ctx, view, y[:, lo:lo + width], out_scale=scale)
+            m.inner(x, ctx, view, y[:, lo:lo + width], out_scale=scale, **kw)
             lo += width
         return self.out.forward_partial(y)
