@@ -386,6 +386,43 @@ def fogurax_configs(size, layers=None):
     return fogurax, veterax
 
 
+# ---- Gopevik beside Fogurax at equal layer sizes ----------------------------------------------------------------------
+# Eight layers in turn: block-masked attention beside retention, and the gated delta rule, every one with a dense gated
+# feed-forward.  Attention heads of 128 with values of 128 and blocks of 1,024 positions, width / 64 retention heads of 64, delta
+# heads of 128 with values of 128 (two value heads to a query/key head, their values twice the width together), norms in 8 parts.
+# The other model: Fogurax (the closest one: the same attention kernels, a recurrent mixer with a matrix state per head beside
+# attention) with the same width, depth, heads, recurrent heads of 64, dense feed-forward and vocabulary: windowed attention
+# beside the recurrent mixer, and convolved attention, in turn.
+GOPEVIK_SIZES = {
+    "S": dict(width=2048, vocab=32000, heads=(16, 2), dim=128, span=1024, ff=5632),
+    "M": dict(width=4096, vocab=32000, heads=(32, 8), dim=128, span=1024, ff=11008),
+}
+
+
+def gopevik_configs(size, layers=None):
+    from qwen_decoder_b200.config import config_from_dict
+    z = GOPEVIK_SIZES[size]
+    (H, G), d, n = z["heads"], z["dim"], z["width"] // 64
+    base = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    count = max(1, layers or 8)     # fewer layers of the same sizes: a capture under a profiler holds fewer weights
+    both = {"type": "parallel", "mlp": dense, "mixer": {
+        "left": dict(base, mask={"size": z["span"]}, rot={"base": 200000.0, "dims": d, "scaling": {"factor": 4.0}}),
+        "right": {"heads": n, "dim": 64, "vdim": 64, "decay": [1.0 - 2.0 ** (-3.0 - 6.0 * i / n) for i in range(n)],
+                  "rot": {"base": 10000.0, "dims": 64}},
+        "left_scale": 0.8, "right_scale": 1.25}}
+    delta = {"type": "delta", "mlp": dense, "mixer": {"heads": z["width"] // 64, "kv_heads": z["width"] // 128, "dim": 128, "vdim": 128, "conv": 4}}
+    gopevik = config_from_dict({"architecture": "Gopevik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5, "groups": 8},
+                                "layers": ([both, delta] * 4)[:count]})
+    conv = {"type": "attention", "mlp": dense, "mixer": dict(base, conv=4, rot={"base": 200000.0, "dims": d})}
+    mixed = {"type": "parallel", "mlp": dense, "mixer": {
+        "left": dict(base, mask={"size": z["span"]}, rot={"base": 10000.0, "dims": d}),
+        "right": {"heads": n, "dim": 64, "rank": 64}, "left_scale": 0.8, "right_scale": 1.25}}
+    fogurax = config_from_dict({"architecture": "Fogurax", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+                                "layers": ([mixed, conv] * 4)[:count]})
+    return gopevik, fogurax
+
+
 def hybrid_bench(args, label="hybrid", configs=None, other="dense"):
     """``--micro hybrid`` (and ``--micro veterax``, which passes its own pair of models): decode steps (batch 1, 8, 64 at ``--context``) and a prompt of ``--prefill-tokens`` tokens, for the
     hybrid design and for the dense decoder at equal sizes; one JSON line.  ``--only hybrid|dense`` and ``--phase`` narrow it
@@ -537,6 +574,8 @@ def micro(args):
         return hybrid_bench(args, "solopel", lambda size: solopel_configs(size, args.veterax_layers), other="veterax")
     if args.micro == "fogurax":
         return hybrid_bench(args, "fogurax", lambda size: fogurax_configs(size, args.veterax_layers), other="veterax")
+    if args.micro == "gopevik":
+        return hybrid_bench(args, "gopevik", lambda size: gopevik_configs(size, args.veterax_layers), other="fogurax")
     if args.micro == "latent_attend":
         return latent_attend_micro(args)
     """One kernel alone: W-streaming contraction, decode attention or prefill attention at the 3B sizes."""
@@ -788,7 +827,7 @@ def main():
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--timeline", action="store_true",
                     help="with --micro prefill_attention: print the kernel's own time stamps of one CTA (microseconds) to stderr")
-    ap.add_argument("--micro", default=None, choices=["gemm", "decode_attention", "decode_attention_rope", "prefill_attention", "serve", "mixed_step", "hybrid", "latent_attend", "veterax", "solopel", "fogurax"],
+    ap.add_argument("--micro", default=None, choices=["gemm", "decode_attention", "decode_attention_rope", "prefill_attention", "serve", "mixed_step", "hybrid", "latent_attend", "veterax", "solopel", "fogurax", "gopevik"],
                     help="time one kernel alone at the 3B shape (for profiles/), or with 'serve' a whole run of "
                          "--batch requests (--context prompt tokens, --steps new tokens each) through the entry "
                          "point; print one JSON line and exit")
@@ -802,7 +841,7 @@ def main():
     ap.add_argument("--micro-splits", type=int, default=1, help="gemm with --micro-graph: shares of K (partial sums)")
     ap.add_argument("--hybrid-size", default="S", choices=["S", "M"], help="hybrid, veterax, solopel: which layer sizes")
     ap.add_argument("--only", default=None, choices=["hybrid", "dense", "other"], help="hybrid, veterax, solopel: one of the two models (hybrid = the first; dense, other = the second)")
-    ap.add_argument("--veterax-layers", type=int, default=None, help="veterax, solopel: fewer layers than the size has")
+    ap.add_argument("--veterax-layers", type=int, default=None, help="veterax, solopel, fogurax, gopevik: fewer layers than the size has")
     ap.add_argument("--phase", default="all", choices=["all", "decode", "prefill"], help="hybrid: decode steps, the prompt, or both")
     ap.add_argument("--history", type=int, default=2048, help="mixed_step: cached tokens before the prompt portion")
     ap.add_argument("--stamps", action="store_true",
