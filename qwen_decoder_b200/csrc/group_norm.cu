@@ -43,6 +43,116 @@ __device__ __forceinline__ void group_factors(const float* sq, int n, int groups
   __syncthreads();
 }
 
+// Four neighbouring elements of the branch's output: its partial sums added up, and its bias.
+__device__ __forceinline__ float4 delta4(const GroupNorm& a, size_t s, int i, float4 bias) {
+  float4 d;
+  if (a.delta_dtype == QD_F32) {
+    const float4* dp = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(a.delta) + s * a.D) + i;
+    d = *dp;
+    for (int p = 1; p < a.n_parts; p++) {
+      const float4 e = dp[p * (a.part_stride >> 2)];
+      d.x += e.x; d.y += e.y; d.z += e.z; d.w += e.w;
+    }
+  } else {
+    const uint2 raw = reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(a.delta) + s * a.D)[i];
+    const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&raw.x);
+    const __nv_bfloat162 hi = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
+    d = make_float4(__low2float(lo), __high2float(lo), __low2float(hi), __high2float(hi));
+  }
+  return make_float4(d.x + bias.x, d.y + bias.y, d.z + bias.z, d.w + bias.w);
+}
+__device__ __forceinline__ void out4(const GroupNorm& a, size_t r, int i, float4 o) {
+  if (a.out_dtype == QD_F32) {
+    reinterpret_cast<float4*>(reinterpret_cast<float*>(a.out) + r * a.D)[i] = o;
+    return;
+  }
+  __nv_bfloat162 lo = __floats2bfloat162_rn(o.x, o.y), hi = __floats2bfloat162_rn(o.z, o.w);
+  uint2 raw;
+  raw.x = *reinterpret_cast<unsigned*>(&lo);
+  raw.y = *reinterpret_cast<unsigned*>(&hi);
+  reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + r * a.D)[i] = raw;
+}
+__device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// ------------------------------------------------------------------------------------- parts of whole warps
+// Every part of D a multiple of 128 elements: the 32 float4 that a warp holds at one turn lie in one part, so a norm costs
+// one meeting of the CTA -- every warp leaves its sum, and adds up its part's sums itself.
+template <int VPT, int MAX_THREADS>
+__global__ void __launch_bounds__(MAX_THREADS)
+group_add_norm_warp_kernel(GroupNorm a) {
+  pdl_launch_dependents();
+  extern __shared__ float gn_sm[];                    // [D / 128] sums of each norm
+  const int n4 = a.D >> 2, lane = threadIdx.x & 31;
+  float4 wp[VPT], wn[VPT], bias[VPT], v[VPT], xv[VPT];
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int q = 0; q < VPT; q++) {                     // no kernel of a step writes these
+    const int i = threadIdx.x + q * blockDim.x;
+    wp[q] = (a.post_w && i < n4) ? reinterpret_cast<const float4*>(a.post_w)[i] : zero;
+    wn[q] = (a.pre_w && i < n4) ? reinterpret_cast<const float4*>(a.pre_w)[i] : zero;
+    bias[q] = (a.delta_bias && i < n4) ? reinterpret_cast<const float4*>(a.delta_bias)[i] : zero;
+  }
+  pdl_wait();
+  const int r = blockIdx.x;
+  const size_t s = a.rows ? (size_t)a.rows[r] : (size_t)r;
+  float4* xr = reinterpret_cast<float4*>(a.x + s * a.D);
+  float* sums = gn_sm;
+  // 1 / sqrt(mean over the part of this warp's float4 ``i`` + eps)
+  auto factor = [&](int i, int part4, float eps) {
+    const int g0 = i / part4 * (part4 >> 5);
+    float t = 0.f;
+    for (int k = lane; k < part4 >> 5; k += 32) t += sums[g0 + k];
+    return 1.0f / sqrtf(warp_sum(t) / (float)(4 * part4) + eps);
+  };
+#pragma unroll
+  for (int q = 0; q < VPT; q++) {
+    const int i = threadIdx.x + q * blockDim.x;
+    xv[q] = v[q] = zero;
+    if (i < n4) {
+      xv[q] = xr[i];
+      if (a.delta) v[q] = delta4(a, s, i, bias[q]);
+    }
+  }
+  if (a.delta && a.post_w) {
+#pragma unroll
+    for (int q = 0; q < VPT; q++) {
+      const int i = threadIdx.x + q * blockDim.x;
+      const float t = warp_sum(sq4(v[q]));
+      if (lane == 0 && i < n4) sums[i >> 5] = t;
+    }
+    __syncthreads();
+    const int part4 = n4 / a.post_groups;
+#pragma unroll
+    for (int q = 0; q < VPT; q++) {
+      const int i = threadIdx.x + q * blockDim.x;
+      if (i >= n4) continue;                          // whole warps: D is a multiple of 128
+      const float c = factor(i, part4, a.post_eps);
+      v[q] = make_float4(v[q].x * c * wp[q].x, v[q].y * c * wp[q].y, v[q].z * c * wp[q].z, v[q].w * c * wp[q].w);
+    }
+  }
+  sums = gn_sm + (n4 >> 5);
+#pragma unroll
+  for (int q = 0; q < VPT; q++) {
+    const int i = threadIdx.x + q * blockDim.x;
+    xv[q].x += v[q].x; xv[q].y += v[q].y; xv[q].z += v[q].z; xv[q].w += v[q].w;
+    if (a.delta && a.write_back && i < n4) xr[i] = xv[q];
+    if (a.pre_w) {
+      const float t = warp_sum(sq4(xv[q]));
+      if (lane == 0 && i < n4) sums[i >> 5] = t;
+    }
+  }
+  if (!a.pre_w) return;
+  __syncthreads();
+  const int part4 = n4 / a.pre_groups;
+#pragma unroll
+  for (int q = 0; q < VPT; q++) {
+    const int i = threadIdx.x + q * blockDim.x;
+    if (i >= n4) continue;
+    const float c = factor(i, part4, a.pre_eps);
+    out4(a, (size_t)r, i, make_float4(xv[q].x * c * wn[q].x, xv[q].y * c * wn[q].y, xv[q].z * c * wn[q].z, xv[q].w * c * wn[q].w));
+  }
+}
+
 // ------------------------------------------------------------------------------------- four elements at a time
 // D and the parts multiples of 4, every pointer 16-byte aligned, D <= 4 * VPT * blockDim.
 template <int VPT>
@@ -76,22 +186,8 @@ group_add_norm_vec_kernel(GroupNorm a) {
     if (i >= n4) continue;
     xv[q] = xr[i];
     if (!a.delta) continue;
-    float4 d;
-    if (a.delta_dtype == QD_F32) {
-      const float4* dp = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(a.delta) + s * a.D) + i;
-      d = *dp;
-      for (int p = 1; p < a.n_parts; p++) {
-        const float4 e = dp[p * (a.part_stride >> 2)];
-        d.x += e.x; d.y += e.y; d.z += e.z; d.w += e.w;
-      }
-    } else {
-      const uint2 raw = reinterpret_cast<const uint2*>(reinterpret_cast<const bf16*>(a.delta) + s * a.D)[i];
-      const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&raw.x);
-      const __nv_bfloat162 hi = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
-      d = make_float4(__low2float(lo), __high2float(lo), __low2float(hi), __high2float(hi));
-    }
-    v[q] = make_float4(d.x + bias[q].x, d.y + bias[q].y, d.z + bias[q].z, d.w + bias[q].w);
-    if (a.post_w) sq[i] = v[q].x * v[q].x + v[q].y * v[q].y + v[q].z * v[q].z + v[q].w * v[q].w;
+    v[q] = delta4(a, s, i, bias[q]);
+    if (a.post_w) sq[i] = sq4(v[q]);
   }
   const int post_part4 = n4 / a.post_groups, pre_part4 = n4 / a.pre_groups;
   if (a.delta && a.post_w) group_factors(sq, n4, a.post_groups, post_part4 * 4, a.post_eps, scratch, f);
@@ -107,7 +203,7 @@ group_add_norm_vec_kernel(GroupNorm a) {
       xv[q].x += v[q].x; xv[q].y += v[q].y; xv[q].z += v[q].z; xv[q].w += v[q].w;
       if (a.write_back) xr[i] = xv[q];
     }
-    if (a.pre_w) sq[i] = xv[q].x * xv[q].x + xv[q].y * xv[q].y + xv[q].z * xv[q].z + xv[q].w * xv[q].w;
+    if (a.pre_w) sq[i] = sq4(xv[q]);
   }
   if (!a.pre_w) return;
   group_factors(sq, n4, a.pre_groups, pre_part4 * 4, a.pre_eps, scratch, f);
@@ -116,16 +212,7 @@ group_add_norm_vec_kernel(GroupNorm a) {
     const int i = threadIdx.x + q * blockDim.x;
     if (i >= n4) continue;
     const float c = f[i / pre_part4];
-    const float4 o = make_float4(xv[q].x * c * wn[q].x, xv[q].y * c * wn[q].y, xv[q].z * c * wn[q].z, xv[q].w * c * wn[q].w);
-    if (a.out_dtype == QD_F32) {
-      reinterpret_cast<float4*>(reinterpret_cast<float*>(a.out) + (size_t)r * a.D)[i] = o;
-    } else {
-      __nv_bfloat162 lo = __floats2bfloat162_rn(o.x, o.y), hi = __floats2bfloat162_rn(o.z, o.w);
-      uint2 raw;
-      raw.x = *reinterpret_cast<unsigned*>(&lo);
-      raw.y = *reinterpret_cast<unsigned*>(&hi);
-      reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + (size_t)r * a.D)[i] = raw;
-    }
+    out4(a, (size_t)r, i, make_float4(xv[q].x * c * wn[q].x, xv[q].y * c * wn[q].y, xv[q].z * c * wn[q].z, xv[q].w * c * wn[q].w));
   }
 }
 
@@ -194,7 +281,21 @@ extern "C" int qd_group_add_norm(float* x, const void* delta, int delta_dtype, i
   const uintptr_t all = (uintptr_t)x | (uintptr_t)delta | (uintptr_t)delta_bias | (uintptr_t)post_w | (uintptr_t)pre_w |
                         (uintptr_t)out;
   if ((D / post_groups) % 4 == 0 && (D / pre_groups) % 4 == 0 && !(all & 15) && part_stride % 4 == 0 && D <= 16384) {
-    const int n4 = D / 4, threads = n4 < 1024 ? (n4 + 31) / 32 * 32 : 1024;
+    const int n4 = D / 4;
+    if ((D / post_groups) % 128 == 0 && (D / pre_groups) % 128 == 0) {
+      const size_t smem = (size_t)2 * (n4 / 32) * sizeof(float);
+      // few rows: one piece a thread; many rows: two or four, so that more rows are under way
+      if (n4 <= 256) qd_launch(group_add_norm_warp_kernel<1, 256>, dim3(n_rows), dim3(n4), smem, stream, a);
+      else if (n4 <= 512 && n_rows > 128)
+        qd_launch(group_add_norm_warp_kernel<2, 256>, dim3(n_rows), dim3((n4 / 2 + 31) / 32 * 32), smem, stream, a);
+      else if (n4 <= 1024 && n_rows > 128)
+        qd_launch(group_add_norm_warp_kernel<4, 256>, dim3(n_rows), dim3((n4 / 4 + 31) / 32 * 32), smem, stream, a);
+      else if (n4 <= 1024) qd_launch(group_add_norm_warp_kernel<1, 1024>, dim3(n_rows), dim3(n4), smem, stream, a);
+      else if (n4 <= 2048) qd_launch(group_add_norm_warp_kernel<2, 1024>, dim3(n_rows), dim3((n4 / 2 + 31) / 32 * 32), smem, stream, a);
+      else qd_launch(group_add_norm_warp_kernel<4, 1024>, dim3(n_rows), dim3((n4 / 4 + 31) / 32 * 32), smem, stream, a);
+      return qd_last_error();
+    }
+    const int threads = n4 < 1024 ? (n4 + 31) / 32 * 32 : 1024;
     const int most = groups > threads / 32 ? groups : threads / 32;
     const size_t smem = ((size_t)n4 + 2 * most) * sizeof(float);          // at most 4,096 * 3 floats
     if (smem > 48 * 1024) return QD_ERR_UNSUPPORTED;

@@ -16,8 +16,8 @@
 //   finish   out[t, h] = o / sqrt(mean(o^2) + eps) (* norm [dv]) * silu(gate) * out_scale, rounded once
 //   step     scan and finish of single tokens, one per request, in one launch: a CTA owns a whole head
 //
-// Everything is float32 until ``finish``'s store.  The recurrence runs in the order of the tokens with a fixed order of
-// additions, so a portion at once and token by token agree up to how the compiler contracts the same expressions.
+// Everything is float32 until ``finish``'s store.  The order of every sum depends on the sizes and on a token's place in its
+// portion only: however a prompt is cut, the results agree up to the rounding of float32 sums.
 #include "common.cuh"
 #include "short_conv.cuh"
 #include <math.h>
@@ -32,7 +32,7 @@ __device__ __forceinline__ float ls_softplus(float z) { return z > 20.0f ? z : l
 // ------------------------------------------------------------------------------------------------------------ prep
 #define LP_THREADS 128
 #define LP_VCH 128            // channels of v a CTA takes
-#define LP_MAX_TOKENS 8
+#define LP_MAX_TOKENS 16
 
 struct LinearPrep {
   const float* u; long long ld;
@@ -53,17 +53,33 @@ __global__ void __launch_bounds__(LP_THREADS)
 linear_prep_kernel(LinearPrep a) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float lp_sm[];                    // [tokens][d], then [tokens] factors
+  extern __shared__ float lp_sm[];                    // [tokens][d] outputs, [tokens] factors, then the inputs' rows
   const int slot = blockIdx.x, t0 = blockIdx.y * a.tokens, nt = min(a.tokens, a.T - t0);
   const int tid = threadIdx.x;
   const int nq = a.G * a.d, C = 2 * nq + a.H * a.dv;
-  auto channel = [&](int t, int c) {                  // what channel c of the stacked q | k | v is after conv and silu
-    if (a.taps <= 0) return a.u[(size_t)t * a.ld + c];
-    const int r = a.token_req[t];
+  const int back = a.taps > 1 ? a.taps - 1 : 0, first = max(0, t0 - back);     // the rows of u this CTA's tokens read
+  float* rows = lp_sm + (size_t)a.tokens * a.d + a.tokens;
+  // Columns c0 .. c0 + n - 1 of those rows into shared memory, ``w`` apart.
+  auto fetch = [&](int c0, int n, int w) {
+    for (int e = tid; e < (t0 + nt - first) * w; e += LP_THREADS) {
+      const int rr = e / w, c = e - rr * w;
+      if (c < n) rows[e] = a.u[(size_t)(first + rr) * a.ld + c0 + c];
+    }
+    __syncthreads();
+  };
+  // What channel c0 + c of the stacked q | k | v is after convolution and silu, from the fetched rows.
+  auto channel = [&](int t, int c0, int c, int w) {
+    if (a.taps <= 0) return rows[(t - first) * w + c];
+    const int r = a.token_req[t], begin = a.cu_tokens[r], li = t - begin, ch = c0 + c;
     float* kept = a.taps > 1 ? a.state + (size_t)a.slots[r] * a.state_stride + a.conv_off : nullptr;
-    const float y = short_conv_at(a.u, a.ld, C, a.taps, a.conv_w, kept, a.cu_tokens[r], t, c);
-    // every request brings one token: this thread alone reads and writes channel c of its request's kept inputs
-    if (a.advance) short_conv_advance(a.u, a.ld, C, a.taps, kept, t, t + 1, c);
+    float y = 0.f;
+    for (int j = 0; j < a.taps; j++) {
+      const int s = li - (a.taps - 1) + j;            // the tap's place in the portion; before it: a kept input
+      const float v = s >= 0 ? rows[(begin + s - first) * w + c] : kept[(size_t)(a.taps - 1 + s) * C + ch];
+      y = fmaf(a.conv_w[(size_t)ch * a.taps + j], v, y);
+    }
+    // every request brings one token: this thread alone reads and writes the channel's kept inputs of its request
+    if (a.advance) short_conv_advance(a.u, a.ld, C, a.taps, kept, t, t + 1, ch);
     return ls_silu(y);
   };
   if (slot >= 2 * a.G + a.v_slots) {                  // the gates
@@ -77,18 +93,20 @@ linear_prep_kernel(LinearPrep a) {
   }
   if (slot >= 2 * a.G) {                              // channels of v
     const int c0 = (slot - 2 * a.G) * LP_VCH, n = min(LP_VCH, a.H * a.dv - c0);
+    fetch(2 * nq + c0, n, LP_VCH);
     for (int e = tid; e < nt * LP_VCH; e += LP_THREADS) {
       const int tt = e / LP_VCH, c = e - tt * LP_VCH;
-      if (c < n) a.v[(size_t)(t0 + tt) * a.H * a.dv + c0 + c] = channel(t0 + tt, 2 * nq + c0 + c);
+      if (c < n) a.v[(size_t)(t0 + tt) * a.H * a.dv + c0 + c] = channel(t0 + tt, 2 * nq + c0, c, LP_VCH);
     }
     return;
   }
   const bool is_q = slot < a.G;
   const int head = is_q ? slot : slot - a.G, base = (is_q ? 0 : nq) + head * a.d, d = a.d;
   float* f = lp_sm + (size_t)a.tokens * d;
+  fetch(base, d, d);
   for (int e = tid; e < nt * d; e += LP_THREADS) {
     const int tt = e / d;
-    lp_sm[e] = channel(t0 + tt, base + e - tt * d);
+    lp_sm[e] = channel(t0 + tt, base, e - tt * d, d);
   }
   __syncthreads();
   const int warp = tid >> 5, lane = tid & 31;
@@ -153,15 +171,23 @@ extern "C" int qd_linear_prep(const float* u, long long ld, int T, int n_request
       (rotary_dim > 0 && (!cos_t || !sin_t || !positions)) || (b_off >= 0 && !beta) ||
       (a_off >= 0 && (!g || !A_log || !dt_bias)) || !q || !k || n_requests > 65535)
     return QD_ERR_UNSUPPORTED;
-  const int tokens = T <= 32 ? 1 : T <= 128 ? 2 : LP_MAX_TOKENS;
+  int tokens = T <= 32 ? 1 : T <= 128 ? 2 : LP_MAX_TOKENS;
   const int v_slots = taps > 0 ? (H * dv + LP_VCH - 1) / LP_VCH : 0;
   const int slots_x = 2 * G + v_slots + (b_off >= 0 || a_off >= 0 ? 1 : 0);
-  if ((T + tokens - 1) / tokens > 65535) return QD_ERR_UNSUPPORTED;
+  const int width = v_slots && LP_VCH > d ? LP_VCH : d;
+  auto bytes = [&](int n) { return ((size_t)n * d + n + (size_t)(n + (taps > 1 ? taps - 1 : 0)) * width) * sizeof(float); };
+  while (tokens > 1 && bytes(tokens) > 48 * 1024) tokens /= 2;
+  const size_t smem = bytes(tokens);
+  if (smem > 200 * 1024 || (T + tokens - 1) / tokens > 65535) return QD_ERR_UNSUPPORTED;
+  static size_t raised = 48 * 1024;
+  if (smem > raised) {
+    cudaFuncSetAttribute(linear_prep_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    raised = smem;
+  }
   const int advance = update_state && taps > 1 && T == n_requests;       // single tokens, one per request
   const LinearPrep a = {u, ld, T, H, G, d, dv, DP, taps, conv_w, state, state_stride, conv_off, advance, token_req, cu_tokens,
                         slots, unit, unit_eps, rotary_dim, pairing, cos_t, sin_t, positions, q_scale, k_scale, b_off, a_off,
                         A_log, dt_bias, q, k, v, beta, g, v_slots, tokens};
-  const size_t smem = ((size_t)tokens * d + tokens) * sizeof(float);      // at most 8 * 257 floats
   qd_launch(linear_prep_kernel, dim3(slots_x, (T + tokens - 1) / tokens), dim3(LP_THREADS), smem, stream, a);
   if (update_state && taps > 1 && !advance) {
     const int C = 2 * G * d + H * dv;
@@ -172,88 +198,115 @@ extern "C" int qd_linear_prep(const float* u, long long ld, int T, int n_request
 }
 
 // ------------------------------------------------------------------------------------------------------------ scan
-// Thread (x = tid & 3, column = tid >> 2) keeps the elements i = 16 m + 4 x + c (c < 4, m < NI / 4) of one value
-// column of S in registers; the four threads of a column are neighbouring lanes.
 #define LS_GROUP 16           // tokens of operands in shared memory at a time (two such groups in flight)
-#define LS_COLS 32            // value columns a CTA owns
-#define LS_THREADS (4 * LS_COLS)
 
 struct LinearScan {
   const float *q, *k;                     // [T, G, DP]
   const float* v; long long ldv;          // row t at t * ldv, head h at + h * dv
   const float* g; int g_ld;               // [T, H] (g_ld = H), or one number per head (g_ld = 0)
   const float* beta;                      // [T, H] (delta rule)
+  const float* coef;                      // [T, H, LS_COEF] (delta rule, portions)
   int H, G, d, dv;
   float* state; long long state_stride, s_off; int vec;         // vec: rows of d elements start on 16-byte boundaries
   const int *cu_tokens, *slots;
   int write_state;
 };
 
-template <int NI>
-__device__ __forceinline__ void ls_load_state(float (&s)[NI], const float* col, int x, int d, bool live, bool vec) {
+// Two float32 numbers that one instruction works on (each rounded as by itself).
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 f2_make(float lo, float hi) {
+  f2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float f2_lo(f2 v) { return __uint_as_float((unsigned)v); }
+__device__ __forceinline__ float f2_hi(f2 v) { return __uint_as_float((unsigned)(v >> 32)); }
+// PACKED: one instruction for both; else two (a loop that waits for latencies rather than for issue slots is better off).
+template <bool PACKED>
+__device__ __forceinline__ f2 f2_fma(f2 a, f2 b, f2 c) {
+  if (!PACKED) return f2_make(fmaf(f2_lo(a), f2_lo(b), f2_lo(c)), fmaf(f2_hi(a), f2_hi(b), f2_hi(c)));
+  f2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+template <bool PACKED>
+__device__ __forceinline__ f2 f2_mul(f2 a, f2 b) {
+  if (!PACKED) return f2_make(f2_lo(a) * f2_lo(b), f2_hi(a) * f2_hi(b));
+  f2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ f2 f2_add(f2 a, f2 b) { return f2_make(f2_lo(a) + f2_lo(b), f2_hi(a) + f2_hi(b)); }
+
+// A thread's share of one value column of S: lane x of X takes the E elements i = 4 X m + 4 x + c (c < 4, m < E / 4), two to a
+// register pair.
+template <int E, int X>
+__device__ __forceinline__ void ls_load_state(f2 (&s)[E / 2], const float* col, int x, int d, bool live, bool vec) {
 #pragma unroll
-  for (int m = 0; m < NI / 4; m++) {
-    const int i = 16 * m + 4 * x;
+  for (int m = 0; m < E / 4; m++) {
+    const int i = 4 * X * m + 4 * x;
     if (vec) {
-      const float4 t = live && i < d ? *reinterpret_cast<const float4*>(col + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-      s[4 * m] = t.x; s[4 * m + 1] = t.y; s[4 * m + 2] = t.z; s[4 * m + 3] = t.w;
+      const ulonglong2 t = live && i < d ? *reinterpret_cast<const ulonglong2*>(col + i) : make_ulonglong2(0, 0);
+      s[2 * m] = t.x;
+      s[2 * m + 1] = t.y;
     } else {
 #pragma unroll
-      for (int c = 0; c < 4; c++) s[4 * m + c] = live && i + c < d ? col[i + c] : 0.f;
+      for (int c = 0; c < 2; c++)
+        s[2 * m + c] = f2_make(live && i + 2 * c < d ? col[i + 2 * c] : 0.f, live && i + 2 * c + 1 < d ? col[i + 2 * c + 1] : 0.f);
     }
   }
 }
-template <int NI>
-__device__ __forceinline__ void ls_store_state(const float (&s)[NI], float* col, int x, int d, bool vec) {
+template <int E, int X>
+__device__ __forceinline__ void ls_store_state(const f2 (&s)[E / 2], float* col, int x, int d, bool vec) {
 #pragma unroll
-  for (int m = 0; m < NI / 4; m++) {
-    const int i = 16 * m + 4 * x;
+  for (int m = 0; m < E / 4; m++) {
+    const int i = 4 * X * m + 4 * x;
     if (vec) {
-      if (i < d) *reinterpret_cast<float4*>(col + i) = make_float4(s[4 * m], s[4 * m + 1], s[4 * m + 2], s[4 * m + 3]);
+      if (i < d) *reinterpret_cast<ulonglong2*>(col + i) = make_ulonglong2(s[2 * m], s[2 * m + 1]);
     } else {
 #pragma unroll
-      for (int c = 0; c < 4; c++)
-        if (i + c < d) col[i + c] = s[4 * m + c];
+      for (int c = 0; c < 2; c++) {
+        if (i + 2 * c < d) col[i + 2 * c] = f2_lo(s[2 * m + c]);
+        if (i + 2 * c + 1 < d) col[i + 2 * c + 1] = f2_hi(s[2 * m + c]);
+      }
     }
   }
 }
 
-// One token: the state moves on, and this thread's share of S^T q comes back.  kr / qr: the token's k and q (DP elements,
-// 16-byte aligned).
-template <int NI, bool DELTA>
-__device__ __forceinline__ float ls_token(float (&s)[NI], const float* kr, const float* qr, float v, float g, float beta, int x) {
-  float4 kk[NI / 4];
+// This thread's share of S^T k of a column: s . k over its elements.
+template <int E, bool PACKED>
+__device__ __forceinline__ float ls_dot(const f2 (&s)[E / 2], const f2 (&k)[E / 2]) {
+  f2 a = f2_mul<PACKED>(s[0], k[0]), b = f2_mul<PACKED>(s[1], k[1]);
 #pragma unroll
-  for (int m = 0; m < NI / 4; m++) kk[m] = *reinterpret_cast<const float4*>(kr + 16 * m + 4 * x);
-  float w = v;
-  if (DELTA) {
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-    for (int m = 0; m < NI / 4; m++) {
-      a.x = fmaf(s[4 * m], kk[m].x, a.x);
-      a.y = fmaf(s[4 * m + 1], kk[m].y, a.y);
-      a.z = fmaf(s[4 * m + 2], kk[m].z, a.z);
-      a.w = fmaf(s[4 * m + 3], kk[m].w, a.w);
-    }
-    float dot = (a.x + a.y) + (a.z + a.w);
-    dot += __shfl_xor_sync(0xffffffffu, dot, 2);
-    dot += __shfl_xor_sync(0xffffffffu, dot, 1);
-    w = beta * fmaf(-g, dot, v);                      // (g S)^T k = g (S^T k)
+  for (int m = 1; m < E / 4; m++) {
+    a = f2_fma<PACKED>(s[2 * m], k[2 * m], a);
+    b = f2_fma<PACKED>(s[2 * m + 1], k[2 * m + 1], b);
   }
-  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+  a = f2_add(a, b);
+  return f2_lo(a) + f2_hi(a);
+}
+// s <- g s + w k
+template <int E, bool PACKED>
+__device__ __forceinline__ void ls_move(f2 (&s)[E / 2], const f2 (&k)[E / 2], float w, float g) {
+  const f2 ww = f2_make(w, w), gg = f2_make(g, g);
 #pragma unroll
-  for (int m = 0; m < NI / 4; m++) {
-    const float4 qq = *reinterpret_cast<const float4*>(qr + 16 * m + 4 * x);
-    s[4 * m] = fmaf(kk[m].x, w, g * s[4 * m]);
-    s[4 * m + 1] = fmaf(kk[m].y, w, g * s[4 * m + 1]);
-    s[4 * m + 2] = fmaf(kk[m].z, w, g * s[4 * m + 2]);
-    s[4 * m + 3] = fmaf(kk[m].w, w, g * s[4 * m + 3]);
-    o.x = fmaf(s[4 * m], qq.x, o.x);
-    o.y = fmaf(s[4 * m + 1], qq.y, o.y);
-    o.z = fmaf(s[4 * m + 2], qq.z, o.z);
-    o.w = fmaf(s[4 * m + 3], qq.w, o.w);
+  for (int m = 0; m < E / 2; m++) s[m] = f2_fma<PACKED>(k[m], ww, f2_mul<PACKED>(gg, s[m]));
+}
+// s <- s + w k
+template <int E, bool PACKED>
+__device__ __forceinline__ void ls_add(f2 (&s)[E / 2], const f2 (&k)[E / 2], float w) {
+  const f2 ww = f2_make(w, w);
+#pragma unroll
+  for (int m = 0; m < E / 2; m++) s[m] = f2_fma<PACKED>(k[m], ww, s[m]);
+}
+template <int E, int X>
+__device__ __forceinline__ void ls_row(f2 (&r)[E / 2], const float* row, int x) {
+#pragma unroll
+  for (int m = 0; m < E / 4; m++) {
+    const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(row + 4 * X * m + 4 * x);
+    r[2 * m] = t.x;
+    r[2 * m + 1] = t.y;
   }
-  return (o.x + o.y) + (o.z + o.w);
 }
 
 __device__ __forceinline__ void ls_cp16(float* smem, const float* gmem, bool there) {
@@ -265,85 +318,284 @@ __device__ __forceinline__ void ls_cp4(float* smem, const float* gmem, bool ther
                "r"(there ? 4 : 0));
 }
 
-// grid (ceil(dv / LS_COLS), H, requests).  out float32 [T, H * dv] dense.
-template <int NI, bool DELTA>
-__global__ void __launch_bounds__(LS_THREADS)
+// X lanes that hold X partial sums each (acc[0 .. X - 1]) add them up: after the step with distance o a lane keeps the o sums of
+// the half that its bit o of x names, and lane x ends with sum x -- the same tree of additions for every sum.
+template <int X>
+__device__ __forceinline__ float ls_reduce(float (&acc)[X], int x) {
+#pragma unroll
+  for (int o = X / 2; o > 0; o >>= 1) {
+    const bool upper = x & o;
+#pragma unroll
+    for (int i = 0; i < o; i++) {
+      const float send = upper ? acc[i] : acc[i + o], keep = upper ? acc[i + o] : acc[i];
+      acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+    }
+  }
+  return acc[0];
+}
+
+#define LS_COEF 12            // numbers per (token, head) of the delta rule's runs
+// What a stage of shared memory holds of LS_GROUP tokens: q, k [LS_GROUP][DP], v [LS_GROUP][COLS] and the decays [LS_GROUP], or
+// with the delta rule its coefficients [LS_GROUP][LS_COEF].
+template <int DP, bool DELTA, int COLS>
+struct LsStage {
+  static constexpr int Q = 0, K = LS_GROUP * DP, V = K + LS_GROUP * DP, G = V + LS_GROUP * COLS,
+                       FLOATS = G + LS_GROUP * (DELTA ? LS_COEF : 1);
+};
+
+// Starts the copies of the tokens tb .. tb + LS_GROUP - 1 of a portion that ends at t1.  Places past its end hold q = k = v = 0, a
+// decay of 1 and coefficients of 0 (with 1 for the decays among them), which leave the state as it is.
+template <int DP, bool DELTA, int COLS, int THREADS>
+__device__ __forceinline__ void ls_fetch(const LinearScan& a, float* st, int tb, int t1, int h, int gk, int j0) {
+  using L = LsStage<DP, DELTA, COLS>;
+  const int tid = threadIdx.x;
+#pragma unroll
+  for (int e = tid; e < LS_GROUP * (DP / 4); e += THREADS) {
+    const int tt = e / (DP / 4), c = (e - tt * (DP / 4)) * 4;
+    const bool there = tb + tt < t1;
+    const size_t src = there ? ((size_t)(tb + tt) * a.G + gk) * DP + c : 0;
+    ls_cp16(st + L::Q + tt * DP + c, a.q + src, there);
+    ls_cp16(st + L::K + tt * DP + c, a.k + src, there);
+  }
+#pragma unroll
+  for (int e = tid; e < LS_GROUP * COLS; e += THREADS) {
+    const int tt = e / COLS, c = e - tt * COLS;
+    const bool there = tb + tt < t1 && j0 + c < a.dv;
+    ls_cp4(st + L::V + e, there ? a.v + (size_t)(tb + tt) * a.ldv + (size_t)h * a.dv + j0 + c : a.v, there);
+  }
+  if (DELTA) {
+    if (tid < LS_GROUP * (LS_COEF / 4)) {
+      const int tt = tid / (LS_COEF / 4), c = tid - tt * (LS_COEF / 4);
+      float* dst = st + L::G + tt * LS_COEF + 4 * c;
+      if (tb + tt < t1) ls_cp16(dst, a.coef + ((size_t)(tb + tt) * a.H + h) * LS_COEF + 4 * c, true);
+      else *reinterpret_cast<float4*>(dst) = c == 2 ? make_float4(a.coef[((size_t)(t1 - 1) * a.H + h) * LS_COEF + 8], 1.f, 0.f, 0.f)
+                                                    : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  } else if (tid < LS_GROUP) {
+    if (tb + tid < t1) ls_cp4(st + L::G + tid, a.g + (a.g_ld ? (size_t)(tb + tid) * a.g_ld : 0) + h, true);
+    else st[L::G + tid] = 1.0f;
+  }
+  asm volatile("cp.async.commit_group;\n" ::);
+}
+
+// Without the delta rule: grid (ceil(dv / COLS), H, requests); eight neighbouring lanes share CPT neighbouring value columns (a
+// thread reads its part of k and q once for all of them); token by token.  out float32 [T, H * dv] dense.
+template <int DP, int COLS, int CPT>
+__global__ void __launch_bounds__(8 * COLS / CPT)
 linear_scan_kernel(LinearScan a, float* __restrict__ out) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int DP = 4 * NI, STAGE = LS_GROUP * (2 * DP + LS_COLS + 2);
-  extern __shared__ __align__(16) float ls_sm[];      // two stages of [q][k][v][g][beta]
-  const int tid = threadIdx.x, x = tid & 3, jl = tid >> 2;
-  const int h = blockIdx.y, req = blockIdx.z, j0 = blockIdx.x * LS_COLS, j = j0 + jl;
+  using L = LsStage<DP, false, COLS>;
+  constexpr int THREADS = 8 * COLS / CPT, E = DP / 8, RUN = 8 / CPT;
+  extern __shared__ __align__(16) float ls_sm[];      // two stages
+  const int tid = threadIdx.x, x = tid & 7, jl = (tid >> 3) * CPT;
+  const int h = blockIdx.y, req = blockIdx.z, j0 = blockIdx.x * COLS, j = j0 + jl;
   const int gk = h / (a.H / a.G), d = a.d, dv = a.dv;
-  const bool live = j < dv;
   const int t0 = a.cu_tokens[req], t1 = a.cu_tokens[req + 1];
   if (t0 >= t1) return;
-  float* col = a.state + (size_t)a.slots[req] * a.state_stride + a.s_off + ((size_t)h * dv + (live ? j : 0)) * d;
-  float s[NI];
-  // Operands of the tokens tb .. tb + LS_GROUP - 1; places past the portion's end hold q = k = v = beta = 0 and g = 1,
-  // which leave the state as it is.
-  auto fetch = [&](int tb, int stage) {
-    float* qs = ls_sm + stage * STAGE;
-    float* ks = qs + LS_GROUP * DP;
-    float* vs = ks + LS_GROUP * DP;
-    float* gs = vs + LS_GROUP * LS_COLS;
-    float* bs = gs + LS_GROUP;
-    for (int e = tid; e < LS_GROUP * NI; e += LS_THREADS) {
-      const int tt = e / NI, c = (e - tt * NI) * 4;
-      const bool there = tb + tt < t1;
-      const size_t src = there ? ((size_t)(tb + tt) * a.G + gk) * DP + c : 0;
-      ls_cp16(qs + tt * DP + c, a.q + src, there);
-      ls_cp16(ks + tt * DP + c, a.k + src, there);
-    }
-    for (int e = tid; e < LS_GROUP * LS_COLS; e += LS_THREADS) {
-      const int tt = e / LS_COLS, c = e - tt * LS_COLS;
-      const bool there = tb + tt < t1 && j0 + c < dv;
-      ls_cp4(vs + e, there ? a.v + (size_t)(tb + tt) * a.ldv + (size_t)h * dv + j0 + c : a.v, there);
-    }
-    if (tid < LS_GROUP) {
-      const bool there = tb + tid < t1;
-      if (there) ls_cp4(gs + tid, a.g + (a.g_ld ? (size_t)(tb + tid) * a.g_ld : 0) + h, true);
-      else gs[tid] = 1.0f;
-      if (DELTA) ls_cp4(bs + tid, there ? a.beta + (size_t)(tb + tid) * a.H + h : a.beta, there);
-    }
-    asm volatile("cp.async.commit_group;\n" ::);
-  };
-  fetch(t0, 0);
-  ls_load_state<NI>(s, col, x, d, live, a.vec);
+  float* S = a.state + (size_t)a.slots[req] * a.state_stride + a.s_off + (size_t)h * dv * d;
+  ls_fetch<DP, false, COLS, THREADS>(a, ls_sm, t0, t1, h, gk, j0);
+  f2 s[CPT][E / 2];
+#pragma unroll
+  for (int c = 0; c < CPT; c++) ls_load_state<E, 8>(s[c], S + (size_t)(j + c < dv ? j + c : 0) * d, x, d, j + c < dv, a.vec);
   int stage = 0;
   for (int tb = t0; tb < t1; tb += LS_GROUP, stage ^= 1) {
     if (tb + LS_GROUP < t1) {
-      fetch(tb + LS_GROUP, stage ^ 1);
+      ls_fetch<DP, false, COLS, THREADS>(a, ls_sm + (stage ^ 1) * L::FLOATS, tb + LS_GROUP, t1, h, gk, j0);
       asm volatile("cp.async.wait_group 1;\n" ::);
     } else {
       asm volatile("cp.async.wait_group 0;\n" ::);
     }
     __syncthreads();
-    const float* qs = ls_sm + stage * STAGE;
-    const float* ks = qs + LS_GROUP * DP;
-    const float* vs = ks + LS_GROUP * DP;
-    const float* gs = vs + LS_GROUP * LS_COLS;
-    const float* bs = gs + LS_GROUP;
+    const float* st = ls_sm + stage * L::FLOATS;
     const int nt = min(LS_GROUP, t1 - tb);
-    for (int q4 = 0; q4 < nt; q4 += 4) {
-      float acc[4];
+    for (int b = 0; b < nt; b += RUN) {
+      float acc[8];                                   // token b + p, column jl + c: this thread's share at CPT p + c
 #pragma unroll
-      for (int p = 0; p < 4; p++) {
-        const int tt = q4 + p;
-        acc[p] = ls_token<NI, DELTA>(s, ks + tt * DP, qs + tt * DP, vs[tt * LS_COLS + jl], gs[tt], DELTA ? bs[tt] : 0.f, x);
+      for (int p = 0; p < RUN; p++) {
+        const int tt = b + p;
+        f2 kr[E / 2], qr[E / 2];
+        ls_row<E, 8>(kr, st + L::K + tt * DP, x);
+        ls_row<E, 8>(qr, st + L::Q + tt * DP, x);
+        const float g = st[L::G + tt];
+#pragma unroll
+        for (int c = 0; c < CPT; c++) {
+          ls_move<E, false>(s[c], kr, st[L::V + tt * COLS + jl + c], g);
+          acc[CPT * p + c] = ls_dot<E, false>(s[c], qr);
+        }
       }
-      // The four threads of a column add up their shares of four tokens at once; thread x ends with token q4 + x's sum,
-      // by the same tree of additions for every place of a token.
-      const bool hi2 = x & 2, hi1 = x & 1;
-      const float r0 = (hi2 ? acc[2] : acc[0]) + __shfl_xor_sync(0xffffffffu, hi2 ? acc[0] : acc[2], 2);
-      const float r1 = (hi2 ? acc[3] : acc[1]) + __shfl_xor_sync(0xffffffffu, hi2 ? acc[1] : acc[3], 2);
-      const float o = (hi1 ? r1 : r0) + __shfl_xor_sync(0xffffffffu, hi1 ? r0 : r1, 1);
-      if (q4 + x < nt && live) out[(size_t)(tb + q4 + x) * a.H * dv + (size_t)h * dv + j] = o;
+      const float o = ls_reduce<8>(acc, x);
+      const int tt = b + x / CPT, c = j + x % CPT;
+      if (tt < nt && c < dv) out[(size_t)(tb + tt) * a.H * dv + (size_t)h * dv + c] = o;
     }
     __syncthreads();                                  // this stage is overwritten by the next turn's fetch
   }
-  if (a.write_state && live) ls_store_state<NI>(s, col, x, d, a.vec);
+  if (!a.write_state) return;
+#pragma unroll
+  for (int c = 0; c < CPT; c++)
+    if (j + c < dv) ls_store_state<E, 8>(s[c], S + (size_t)(j + c) * d, x, d, a.vec);
+}
+
+// The delta rule in runs of four tokens.  With S0 the state before a run, G_p = g_0 .. g_p and d(s, p) = g_(s+1) .. g_p,
+//   x_p = beta_p (v_p - G_p S0^T k_p - sum_(s < p) d(s, p) (k_s . k_p) x_s)
+//   o_p = G_p S0^T q_p + sum_(s <= p) d(s, p) (k_s . q_p) x_s;        S <- G_3 S0 + sum_s d(s, 3) k_s x_s^T
+// which is the rule token by token written out: the four tokens' products with S0 do not wait for one another, only the
+// small triangular system is solved in order.  A run starts at a multiple of four tokens of the portion.
+//
+// Every number in these sums that does not depend on the state, per (token, head), in ``coef`` [T, H, LS_COEF]: with p the
+// token's place in its run,
+//   beta d(s, p) (k_s . k_p) for s < p [0 .. 2];  beta G_p [3];  d(s, p) (k_s . q_p) for s <= p [4 .. 7];  G_p [8];
+//   d(p, the run's last token) [9];  beta [10]          (zero for later s)
+// A warp per (token, query/key head): the dot products once, then the numbers of the value heads that share it.
+template <int DP>
+__global__ void __launch_bounds__(256)
+linear_coef_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ g, int g_ld,
+                   const float* __restrict__ beta, int T, int H, int G, const int* __restrict__ token_req,
+                   const int* __restrict__ cu_tokens, float* __restrict__ coef) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (item >= (long long)T * G) return;
+  const int t = (int)(item / G), gk = (int)(item - (long long)t * G);
+  const int r = token_req[t], p = (t - cu_tokens[r]) & 3, last = min(3, p + cu_tokens[r + 1] - 1 - t);
+  constexpr int N = DP / 32;
+  float kt[N], qt[N];
+#pragma unroll
+  for (int i = 0; i < N; i++) {
+    kt[i] = k[item * DP + lane + 32 * i];
+    qt[i] = q[item * DP + lane + 32 * i];
+  }
+  float kk[4], kq[4];
+#pragma unroll
+  for (int s = 0; s < 4; s++) {
+    kk[s] = kq[s] = 0.f;
+    if (s > p) continue;                              // the same for the whole warp
+    const float* ks = k + ((size_t)(t - p + s) * G + gk) * DP;
+#pragma unroll
+    for (int i = 0; i < N; i++) {
+      const float y = ks[lane + 32 * i];
+      kk[s] = fmaf(y, kt[i], kk[s]);
+      kq[s] = fmaf(y, qt[i], kq[s]);
+    }
+    kk[s] = warp_sum(kk[s]);
+    kq[s] = warp_sum(kq[s]);
+  }
+  const int per = H / G;
+  for (int i = lane; i < per; i += 32) {
+    const int h = gk * per + i;
+    auto decay = [&](int s) { return g[(g_ld ? (size_t)(t - p + s) * g_ld : 0) + h]; };
+    const float b = beta[(size_t)t * H + h];
+    float A[4] = {0.f, 0.f, 0.f, 0.f}, B[4] = {0.f, 0.f, 0.f, 0.f}, dec = 1.f, to_end = 1.f;
+#pragma unroll
+    for (int s = 3; s >= 0; s--) {
+      if (s > p) continue;
+      if (s < p) {
+        dec *= decay(s + 1);
+        A[s] = b * dec * kk[s];
+      }
+      B[s] = dec * kq[s];
+    }
+    dec *= decay(0);
+    for (int s = p + 1; s <= last; s++) to_end *= decay(s);
+    float4* c = reinterpret_cast<float4*>(coef + ((size_t)t * H + h) * LS_COEF);
+    c[0] = make_float4(A[0], A[1], A[2], b * dec);
+    c[1] = make_float4(B[0], B[1], B[2], B[3]);
+    c[2] = make_float4(dec, to_end, b, 0.f);
+  }
+}
+
+// grid (ceil(dv / COLS), H, requests), 8 COLS threads: X = 8 CPT neighbouring lanes share CPT neighbouring value columns, so that a
+// run's 4 CPT products with k and 4 CPT with q are X sums over X lanes: one exchange adds all of them up.
+template <int DP, int COLS, int CPT>
+__global__ void __launch_bounds__(8 * COLS)
+linear_delta_kernel(LinearScan a, float* __restrict__ out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  using L = LsStage<DP, true, COLS>;
+  constexpr int THREADS = 8 * COLS, X = 8 * CPT, E = DP / X;
+  static_assert(E % 4 == 0, "a lane takes whole pieces of four elements");
+  extern __shared__ __align__(16) float ls_sm[];      // two stages
+  const int tid = threadIdx.x, x = tid % X, jl = tid / X * CPT;
+  const int h = blockIdx.y, req = blockIdx.z, j0 = blockIdx.x * COLS, j = j0 + jl;
+  const int gk = h / (a.H / a.G), d = a.d, dv = a.dv;
+  const int t0 = a.cu_tokens[req], t1 = a.cu_tokens[req + 1];
+  if (t0 >= t1) return;
+  float* S = a.state + (size_t)a.slots[req] * a.state_stride + a.s_off + (size_t)h * dv * d;
+  ls_fetch<DP, true, COLS, THREADS>(a, ls_sm, t0, t1, h, gk, j0);
+  f2 s[CPT][E / 2];
+#pragma unroll
+  for (int c = 0; c < CPT; c++) ls_load_state<E, X>(s[c], S + (size_t)(j + c < dv ? j + c : 0) * d, x, d, j + c < dv, a.vec);
+  // after the exchange: lane x has the product with k (first half) or q (second half) of token xp of a run and column xc
+  const int xp = x / CPT & 3, xc = x % CPT;
+  const bool with_q = x >= 4 * CPT;
+  int stage = 0;
+  for (int tb = t0; tb < t1; tb += LS_GROUP, stage ^= 1) {
+    if (tb + LS_GROUP < t1) {
+      ls_fetch<DP, true, COLS, THREADS>(a, ls_sm + (stage ^ 1) * L::FLOATS, tb + LS_GROUP, t1, h, gk, j0);
+      asm volatile("cp.async.wait_group 1;\n" ::);
+    } else {
+      asm volatile("cp.async.wait_group 0;\n" ::);
+    }
+    __syncthreads();
+    const float* st = ls_sm + stage * L::FLOATS;
+    const int nt = min(LS_GROUP, t1 - tb);
+    for (int b = 0; b < nt; b += 4) {
+      f2 kk[4][E / 2];
+      float acc[X];
+#pragma unroll
+      for (int p = 0; p < 4; p++) {
+        f2 r[E / 2];
+        ls_row<E, X>(kk[p], st + L::K + (b + p) * DP, x);
+        ls_row<E, X>(r, st + L::Q + (b + p) * DP, x);
+#pragma unroll
+        for (int c = 0; c < CPT; c++) {
+          acc[p * CPT + c] = ls_dot<E, true>(s[c], kk[p]);
+          acc[4 * CPT + p * CPT + c] = ls_dot<E, true>(s[c], r);
+        }
+      }
+      const float4* co = reinterpret_cast<const float4*>(st + L::G + b * LS_COEF);      // three pieces a token
+      const float4 mine = co[3 * xp + 2];
+      const float sum = ls_reduce<X>(acc, x);
+      const float rhs = fmaf(-co[3 * xp].w, sum, mine.z * st[L::V + (b + xp) * COLS + jl + xc]);
+      float w[CPT][4];
+#pragma unroll
+      for (int c = 0; c < CPT; c++)
+#pragma unroll
+        for (int p = 0; p < 4; p++) w[c][p] = __shfl_sync(0xffffffffu, rhs, p * CPT + c, X);
+      const float4 A1 = co[3], A2 = co[6], A3 = co[9];
+#pragma unroll
+      for (int c = 0; c < CPT; c++) {
+        w[c][1] = fmaf(-A1.x, w[c][0], w[c][1]);
+        w[c][2] = fmaf(-A2.y, w[c][1], fmaf(-A2.x, w[c][0], w[c][2]));
+        w[c][3] = fmaf(-A3.z, w[c][2], fmaf(-A3.y, w[c][1], fmaf(-A3.x, w[c][0], w[c][3])));
+      }
+      const int tt = b + xp, col = j + xc;
+      if (with_q && tt < nt && col < dv) {
+        const float4 B = co[3 * xp + 1];
+        const bool second = CPT > 1 && xc;            // CPT is 1 or 2
+        float o = mine.x * sum;
+        o = fmaf(B.x, second ? w[CPT - 1][0] : w[0][0], o);
+        o = fmaf(B.y, second ? w[CPT - 1][1] : w[0][1], o);
+        o = fmaf(B.z, second ? w[CPT - 1][2] : w[0][2], o);
+        o = fmaf(B.w, second ? w[CPT - 1][3] : w[0][3], o);
+        out[(size_t)(tb + tt) * a.H * dv + (size_t)h * dv + col] = o;
+      }
+      const float g3 = co[11].x, e0 = co[2].y, e1 = co[5].y, e2 = co[8].y;      // the run's last token needs no decay
+#pragma unroll
+      for (int c = 0; c < CPT; c++) {
+        ls_move<E, true>(s[c], kk[0], w[c][0] * e0, g3);
+        ls_add<E, true>(s[c], kk[1], w[c][1] * e1);
+        ls_add<E, true>(s[c], kk[2], w[c][2] * e2);
+        ls_add<E, true>(s[c], kk[3], w[c][3]);
+      }
+    }
+    __syncthreads();                                  // this stage is overwritten by the next turn's fetch
+  }
+  if (!a.write_state) return;
+#pragma unroll
+  for (int c = 0; c < CPT; c++)
+    if (j + c < dv) ls_store_state<E, X>(s[c], S + (size_t)(j + c) * d, x, d, a.vec);
 }
 
 // ---------------------------------------------------------------------------------------------------------- finish
@@ -354,35 +606,72 @@ struct LinearFinish {
   void* out; int out_dtype; long long out_stride;
 };
 
-// grid (ceil(T * H / 8)), a warp per (token, head).
+// A group of LANES lanes per (token, head).
+template <int LANES>
 __global__ void __launch_bounds__(256)
-linear_finish_kernel(const float* __restrict__ o, int T, int H, int dv, LinearFinish f) {
+linear_finish_kernel(const float* __restrict__ o, int T, int H, int dv, LinearFinish f, int vec) {
   pdl_launch_dependents();
   pdl_wait();
-  const int lane = threadIdx.x & 31;
-  const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (item >= (long long)T * H) return;
+  const int lane = threadIdx.x % LANES;
+  long long item = (long long)blockIdx.x * (256 / LANES) + threadIdx.x / LANES;
+  const bool there = item < (long long)T * H;         // every lane of a warp takes part in the shuffles
+  if (!there) item = 0;
   const int t = (int)(item / H), h = (int)(item - (long long)t * H);
   const float* row = o + (size_t)item * dv;
-  float ss = 0.f;
-  for (int i = lane; i < dv; i += 32) { const float y = row[i]; ss = fmaf(y, y, ss); }
-  const float c = f.out_scale / sqrtf(warp_sum(ss) / (float)dv + f.eps);
   const float* gate = f.gate + (size_t)t * f.gate_ld + (size_t)h * dv;
-  for (int i = lane; i < dv; i += 32)
-    ls_st(f.out, f.out_dtype, (size_t)t * f.out_stride + (size_t)h * dv + i,
-          row[i] * c * (f.norm ? f.norm[i] : 1.0f) * ls_silu(gate[i]));
+  const size_t dst = (size_t)t * f.out_stride + (size_t)h * dv;
+  float ss = 0.f;
+  float4 first = make_float4(0.f, 0.f, 0.f, 0.f);     // this lane's first piece stays in registers
+  if (vec) {
+    for (int i = lane * 4; i < dv; i += LANES * 4) {
+      const float4 y = *reinterpret_cast<const float4*>(row + i);
+      if (i == lane * 4) first = y;
+      ss += y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+    }
+  } else {
+    for (int i = lane; i < dv; i += LANES) { const float y = row[i]; ss = fmaf(y, y, ss); }
+  }
+#pragma unroll
+  for (int s = LANES / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  if (!there) return;
+  const float c = f.out_scale / sqrtf(ss / (float)dv + f.eps);
+  if (vec) {
+    for (int i = lane * 4; i < dv; i += LANES * 4) {
+      const float4 y = i == lane * 4 ? first : *reinterpret_cast<const float4*>(row + i);
+      const float4 z = *reinterpret_cast<const float4*>(gate + i);
+      float4 n = make_float4(c, c, c, c);
+      if (f.norm) {
+        const float4 w = *reinterpret_cast<const float4*>(f.norm + i);
+        n = make_float4(c * w.x, c * w.y, c * w.z, c * w.w);
+      }
+      const float4 r = make_float4(y.x * n.x * ls_silu(z.x), y.y * n.y * ls_silu(z.y), y.z * n.z * ls_silu(z.z), y.w * n.w * ls_silu(z.w));
+      if (f.out_dtype == QD_F32) {
+        *reinterpret_cast<float4*>(reinterpret_cast<float*>(f.out) + dst + i) = r;
+      } else {
+        __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+        uint2 raw;
+        raw.x = *reinterpret_cast<unsigned*>(&lo);
+        raw.y = *reinterpret_cast<unsigned*>(&hi);
+        *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(f.out) + dst + i) = raw;
+      }
+    }
+    return;
+  }
+  for (int i = lane; i < dv; i += LANES)
+    ls_st(f.out, f.out_dtype, dst + i, row[i] * c * (f.norm ? f.norm[i] : 1.0f) * ls_silu(gate[i]));
 }
 
 // ------------------------------------------------------------------------------------------------------------ step
-// grid (H, requests), 4 * (columns at a time) threads, at most 512.  Request r's token is token r.
+// grid (H, requests), 4 * (columns at a time) threads, at most 512: four neighbouring lanes to a value column.  Request r's
+// token is token r.
 #define LS_STEP_THREADS 512
 
-template <int NI, bool DELTA>
+template <int DP, bool DELTA>
 __global__ void __launch_bounds__(LS_STEP_THREADS)
 linear_step_kernel(LinearScan a, LinearFinish f) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int DP = 4 * NI;
+  constexpr int E = DP / 4;
   extern __shared__ float st_sm[];                    // [dv] outputs, then 40 of scratch
   const int tid = threadIdx.x, x = tid & 3, jl = tid >> 2, cols = blockDim.x >> 2;
   const int h = blockIdx.x, t = blockIdx.y, d = a.d, dv = a.dv, gk = h / (a.H / a.G);
@@ -396,17 +685,27 @@ linear_step_kernel(LinearScan a, LinearFinish f) {
     const int j = j0 + jl;
     const bool live = j < dv;
     float* col = S + (size_t)(live ? j : 0) * d;
-    float s[NI];
-    ls_load_state<NI>(s, col, x, d, live, a.vec);
-    const float v = live ? a.v[(size_t)t * a.ldv + (size_t)h * dv + j] : 0.f;
-    float o = ls_token<NI, DELTA>(s, kr, qr, v, g, beta, x);
+    f2 s[E / 2];
+    ls_load_state<E, 4>(s, col, x, d, live, a.vec);
+    float w = live ? a.v[(size_t)t * a.ldv + (size_t)h * dv + j] : 0.f;
+    f2 r[E / 2];
+    ls_row<E, 4>(r, kr, x);
+    if (DELTA) {
+      float dot = ls_dot<E, false>(s, r);
+      dot += __shfl_xor_sync(0xffffffffu, dot, 2);
+      dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+      w = beta * fmaf(-g, dot, w);
+    }
+    ls_move<E, false>(s, r, w, g);
+    ls_row<E, 4>(r, qr, x);
+    float o = ls_dot<E, false>(s, r);
     o += __shfl_xor_sync(0xffffffffu, o, 2);
     o += __shfl_xor_sync(0xffffffffu, o, 1);
     if (live && x == 0) {
       st_sm[j] = o;
       ss = fmaf(o, o, ss);
     }
-    if (a.write_state && live) ls_store_state<NI>(s, col, x, d, a.vec);
+    if (a.write_state && live) ls_store_state<E, 4>(s, col, x, d, a.vec);
   }
   const float c = f.out_scale / sqrtf(block_sum(ss, st_sm + dv) / (float)dv + f.eps);     // meets the writes of st_sm, too
   const float* gate = f.gate + (size_t)t * f.gate_ld + (size_t)h * dv;
@@ -416,58 +715,89 @@ linear_step_kernel(LinearScan a, LinearFinish f) {
 }
 
 // ------------------------------------------------------------------------------------------------------- launchers
-// q, k float32 [T, G, DP], DP the padded head size: the smallest of 16, 32, 48, 64, 96, 128, 256 that holds d; v rows
+// q, k float32 [T, G, DP], DP the padded head size: the smallest of 32, 64, 96, 128, 256 that holds d; v rows
 // ``ldv`` apart; g float32 [T, H] (g_ld = H) or [H] (g_ld = 0); beta float32 [T, H]: the delta rule, or null;
 // state float32 rows ``state_stride`` apart, the heads' matrices [H, dv, d] at ``s_off``; o_buf float32 [T, H * dv]
-// (unused when every request brings one token); gate float32 rows ``gate_ld`` apart; norm float32 [dv] or null.
+// (unused when every request brings one token); coef float32 [T, H, LS_COEF] of scratch for the delta rule (unused then, too); gate float32 rows ``gate_ld`` apart; norm float32 [dv] or null.
 extern "C" int qd_linear_scan(const float* q, const float* k, const float* v, long long ldv, const float* g, int g_ld,
                               const float* beta, int T, int n_requests, int H, int G, int d, int dv, int DP,
                               float* state, long long state_stride, long long s_off, const int* cu_tokens,
                               const int* slots, int write_state, float* o_buf, const float* gate, long long gate_ld,
                               const float* norm, float eps, float out_scale, void* out, int out_dtype,
-                              long long out_stride, cudaStream_t stream) {
+                              long long out_stride, const int* token_req, float* coef, cudaStream_t stream) {
   if (T <= 0 || n_requests <= 0) return 0;
   if (H <= 0 || H > 65535 || n_requests > 65535 || G <= 0 || H % G || d <= 0 || dv <= 0 || dv > 8192 || d > DP ||
-      !state || !gate || (g_ld && g_ld != H) || (out_dtype != QD_F32 && out_dtype != QD_BF16))
+      !state || !gate || (g_ld && g_ld != H) || (beta && T != n_requests && (!coef || ((uintptr_t)coef & 15))) || (out_dtype != QD_F32 && out_dtype != QD_BF16))
     return QD_ERR_UNSUPPORTED;
   const bool single = T == n_requests;                // every request has at least one token
   if (!single && !o_buf) return QD_ERR_UNSUPPORTED;
   if (((uintptr_t)q | (uintptr_t)k) & 15) return QD_ERR_UNSUPPORTED;
   const int vec = d % 4 == 0 && state_stride % 4 == 0 && s_off % 4 == 0 && !((uintptr_t)state & 15);
-  const LinearScan a = {q, k, v, ldv, g, g_ld, beta, H, G, d, dv, state, state_stride, s_off, vec, cu_tokens, slots, write_state};
+  const LinearScan a = {q, k, v, ldv, g, g_ld, beta, coef, H, G, d, dv, state, state_stride, s_off, vec, cu_tokens, slots, write_state};
   const LinearFinish f = {gate, gate_ld, norm, eps, out_scale, out, out_dtype, out_stride};
   const int cols = (dv + 7) / 8 * 8 < LS_STEP_THREADS / 4 ? (dv + 7) / 8 * 8 : LS_STEP_THREADS / 4;
   const size_t step_smem = ((size_t)dv + 40) * sizeof(float);
-#define LS_GO2(NI, DELTA)                                                                                             \
+  // few heads: half as many columns to a CTA, so that more multiprocessors work
+  static int sms = 0;
+  if (!sms) {
+    int dev = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+  }
+  const bool narrow = (long long)((dv + 31) / 32) * H * n_requests * 2 <= sms + sms / 8;
+#define LS_LAUNCH(KERNEL, COLS, THREADS, FLOATS)                                                                     \
+  do {                                                                                                                \
+    const size_t smem = (size_t)(FLOATS) * sizeof(float);                                                             \
+    static bool raised = false;                                                                                       \
+    if (!raised && smem > 48 * 1024) {                                                                                \
+      cudaFuncSetAttribute(KERNEL, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
+      raised = true;                                                                                                  \
+    }                                                                                                                 \
+    /* The scan's CTAs are few and long: launched while the kernel before them still runs they would crowd onto the   \
+       multiprocessors that become free first. */                                                                     \
+    qd_plain_next_launch = true;                                                                                      \
+    qd_launch(KERNEL, dim3((dv + COLS - 1) / COLS, H, n_requests), dim3(THREADS), smem, stream, a, o_buf);             \
+  } while (0)
+#define LS_DELTA(DP)                                                                                                  \
   do {                                                                                                                \
     if (single) {                                                                                                     \
-      qd_launch(linear_step_kernel<NI, DELTA>, dim3(H, n_requests), dim3(4 * cols), step_smem, stream, a, f);         \
-    } else {                                                                                                          \
-      const size_t smem = (size_t)2 * LS_GROUP * (8 * NI + LS_COLS + 2) * sizeof(float);                              \
-      static bool raised = false;                                                                                     \
-      if (!raised && smem > 48 * 1024) {                                                                              \
-        cudaFuncSetAttribute(linear_scan_kernel<NI, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
-        raised = true;                                                                                                \
-      }                                                                                                               \
-      qd_launch(linear_scan_kernel<NI, DELTA>, dim3((dv + LS_COLS - 1) / LS_COLS, H, n_requests), dim3(LS_THREADS), smem, \
-                stream, a, o_buf);                                                                                    \
+      qd_launch(linear_step_kernel<DP, true>, dim3(H, n_requests), dim3(4 * cols), step_smem, stream, a, f);          \
+      break;                                                                                                          \
     }                                                                                                                 \
+    qd_launch(linear_coef_kernel<DP>, dim3((unsigned)(((long long)T * G + 7) / 8)), dim3(256), 0, stream, q, k, g, g_ld, \
+              beta, T, H, G, token_req, cu_tokens, coef);                                                             \
+    constexpr int CPT = DP <= 96 ? 1 : 2;                                                                             \
+    if (narrow) LS_LAUNCH((linear_delta_kernel<DP, 16, CPT>), 16, 128, (2 * LsStage<DP, true, 16>::FLOATS));           \
+    else LS_LAUNCH((linear_delta_kernel<DP, 32, CPT>), 32, 256, (2 * LsStage<DP, true, 32>::FLOATS));                  \
   } while (0)
-#define LS_GO(NI) do { if (beta) LS_GO2(NI, true); else LS_GO2(NI, false); } while (0)
+#define LS_PLAIN(DP)                                                                                                  \
+  do {                                                                                                                \
+    if (single) qd_launch(linear_step_kernel<DP, false>, dim3(H, n_requests), dim3(4 * cols), step_smem, stream, a, f); \
+    else if (narrow) LS_LAUNCH((linear_scan_kernel<DP, 16, 1>), 16, 128, (2 * LsStage<DP, false, 16>::FLOATS));        \
+    else LS_LAUNCH((linear_scan_kernel<DP, 32, 2>), 32, 128, (2 * LsStage<DP, false, 32>::FLOATS));                    \
+  } while (0)
+#define LS_GO(DP) do { if (beta) LS_DELTA(DP); else LS_PLAIN(DP); } while (0)
   switch (DP) {
-    case 16: LS_GO(4); break;
-    case 32: LS_GO(8); break;
-    case 48: LS_GO(12); break;
-    case 64: LS_GO(16); break;
-    case 96: LS_GO(24); break;
-    case 128: LS_GO(32); break;
-    case 256: LS_GO(64); break;
+    case 32: LS_GO(32); break;
+    case 64: LS_GO(64); break;
+    case 96: LS_GO(96); break;
+    case 128: LS_GO(128); break;
+    case 256: LS_GO(256); break;
     default: return QD_ERR_UNSUPPORTED;
   }
 #undef LS_GO
-#undef LS_GO2
-  if (!single)
-    qd_launch(linear_finish_kernel, dim3((unsigned)(((long long)T * H + 7) / 8)), dim3(256), 0, stream, (const float*)o_buf,
-              T, H, dv, f);
+#undef LS_DELTA
+#undef LS_PLAIN
+#undef LS_LAUNCH
+  if (!single) {
+    const int fvec = dv % 4 == 0 && gate_ld % 4 == 0 && out_stride % 4 == 0 &&
+                     !(((uintptr_t)o_buf | (uintptr_t)gate | (uintptr_t)norm) & 15) &&
+                     !((uintptr_t)out & (out_dtype == QD_F32 ? 15 : 7));
+    const long long items = (long long)T * H;
+    if (dv <= 64)
+      qd_launch(linear_finish_kernel<16>, dim3((unsigned)((items + 15) / 16)), dim3(256), 0, stream, (const float*)o_buf, T, H, dv, f, fvec);
+    else
+      qd_launch(linear_finish_kernel<32>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, stream, (const float*)o_buf, T, H, dv, f, fvec);
+  }
   return qd_last_error();
 }

@@ -1435,7 +1435,7 @@ def tm_finish(o: torch.Tensor, g: torch.Tensor, norm: torch.Tensor, H: int, d: i
 
 
 # ------------------------------------------------------------------ linear attention with one decay per head and token
-LINEAR_PADS = (16, 32, 48, 64, 96, 128, 256)      # what a head of queries and keys is padded to
+LINEAR_PADS = (32, 64, 96, 128, 256)      # what a head of queries and keys is padded to
 LINEAR_MAX_VDIM = 8192
 
 
@@ -1505,14 +1505,15 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tens
         _contig(t, n)
     single = T == ctx.num_requests
     o = None if single else torch.empty((T, H * dv), dtype=torch.float32, device=q.device)
+    coef = None if single or beta is None else torch.empty((T, H, 12), dtype=torch.float32, device=q.device)
     _check(library("linear_scan").qd_linear_scan(
         _ptr(q), _ptr(k), _ptr(v), _LL(v.stride(0)), _ptr(g), _I(H if g.dim() == 2 else 0), _ptr(beta), _I(T),
         _I(ctx.num_requests), _I(H), _I(G), _I(d), _I(dv), _I(DP), _ptr(state), _LL(state.stride(0)), _LL(s_off),
         _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _I(1 if write_state else 0), _ptr(o), _ptr(gate), _LL(gate.stride(0)),
-        _ptr(norm), _F(eps), _F(out_scale), _ptr(out), _I(dtype_code(out.dtype)), _LL(out.stride(0)), _stream()),
-        "linear_scan")
+        _ptr(norm), _F(eps), _F(out_scale), _ptr(out), _I(dtype_code(out.dtype)), _LL(out.stride(0)), _ptr(ctx.token_request),
+        _ptr(coef), _stream()), "linear_scan")
     if not single:
-        _launch_count[0] += 1
+        _launch_count[0] += 1 if coef is None else 2
 
 
 # ------------------------------------------------------------------ norms in groups, before and after a branch
