@@ -19,7 +19,8 @@ i // (H / G)):
 Per request, one float32 state row: the heads' matrices S [H, vd, d] (a value column's d numbers side by side), then the
 last ``conv_taps`` - 1 projected rows [q | k | v] before the convolution; a fresh row is zero.  All projections of h are
 one stacked product with float32 sums; everything between them and the rounded input of the output matrix is float32 in
-both engine dtypes (``csrc/linear_scan.cu``).  The recurrence runs token by token in the tokens' order.
+both engine dtypes (``csrc/linear_scan.cu``).  The recurrence runs in the tokens' order, the delta rule of longer portions in
+runs of four tokens (the same rule written out).
 
 ``inner`` computes everything up to the output projection into a tensor the caller gives, times ``out_scale``.
 """
