@@ -11,9 +11,11 @@ from .veterax import VeteraxConfig  # registers Veterax
 from .solopel import SolopelConfig  # registers Solopel
 from .fogurax import FoguraxConfig  # registers Fogurax
 from .gopevik import GopevikConfig  # registers Gopevik
+from .furesun import FuresunConfig  # registers Furesun
 
 __all__ = [
-    "ConfigError", "Qwen2Config", "ZunuvikConfig", "VeteraxConfig", "SolopelConfig", "FoguraxConfig", "GopevikConfig", "read_config_json", "write_config_json", "PART_KINDS",
+    "ConfigError", "Qwen2Config", "ZunuvikConfig", "VeteraxConfig", "SolopelConfig", "FoguraxConfig", "GopevikConfig", "FuresunConfig",
+    "read_config_json", "write_config_json", "PART_KINDS",
     "config_from_dict", "create_part", "describe_model", "known_architectures", "load_config",
     "lookup_architecture", "register_architecture", "register_part", "unregister_architecture",
     "unregister_part", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry",

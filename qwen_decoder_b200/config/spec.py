@@ -63,3 +63,4 @@ class ModelSpec:
     final_norm_prefix: str
     lm_head_tensor: Optional[str]           # None: tied to the embedding
     embedding_scale: float = 1.0            # the embedding row is multiplied by this constant
+    logit_softcap: Optional[float] = None   # c: logits z leave as c tanh(z / c)

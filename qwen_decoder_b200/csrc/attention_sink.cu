@@ -15,7 +15,8 @@
 // ``chunk`` positions (blocks counted from position 0 of the sequence); ``gate`` multiplies head h's output row by
 // sigmoid(gate[t * gate_ld + h]) (float32 logits) or, with ``gate_elem``, element i of it by
 // sigmoid(gate[t * gate_ld + h * vd + i]); ``out_scale`` multiplies it by a constant; ``out_stride`` is the
-// distance between output rows, so that the heads may land in a column range of a wider tensor.
+// distance between output rows, so that the heads may land in a column range of a wider tensor; ``cap`` > 0 replaces a
+// score s by cap * tanh(s / cap).
 //
 // A page of the cache holds the keys [G, page_size, d] and then the values [G, page_size, vd].
 #include "common.cuh"
@@ -32,7 +33,18 @@ struct AttnExtra {
   int gate_elem;          // 1: one logit per output element (h * vd + i), 0: one per head
   float out_scale;
   long long out_stride;   // elements between output rows
+  float cap;              // > 0: a score s becomes cap * tanh(s / cap) before the mask
 };
+
+// tanh to the accuracy of a float32 score: the Maclaurin series where |y| <= 1/4 (its first term left out is below
+// 2e-9 there), 1 - 2 / (e^(2y) + 1) elsewhere (an error of some 1e-7 in absolute terms).
+__device__ __forceinline__ float as_tanh_small(float y) {
+  const float t = y * y;
+  return y * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 62.0f / 2835.0f, -17.0f / 315.0f), 2.0f / 15.0f), -1.0f / 3.0f), 1.0f);
+}
+__device__ __forceinline__ float as_tanh_any(float y) {
+  return 1.0f - __fdividef(2.0f, ts_exp2(y * 2.8853900817779268f) + 1.0f);
+}
 
 // The first key a query at ``pos`` sees.
 __device__ __forceinline__ int as_key_lo(int pos, int window, int chunk) {
@@ -205,6 +217,7 @@ sink_attention_generic_kernel(const T* __restrict__ q, long long q_stride, T* __
       float acc = 0.0f;
       for (int i = 0; i < d; i++) acc = fmaf(qs[i], to_float(kr[i]), acc);
       s = acc * scale;
+      if (ex.cap > 0.f) s = ex.cap * tanhf(s / ex.cap);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float c = expf(m - m_new);  // m = -inf on the first tile gives 0
@@ -251,14 +264,14 @@ extern "C" int qd_sink_attention_generic(const void* q, long long q_stride, void
                                          const int* token_req, const int* positions, int n_tokens, int H, int G, int d,
                                          int vd, int page_size, float scale, int window, const float* sinks,
                                          int chunk, const float* gate, long long gate_ld, int gate_elem,
-                                         float out_scale, cudaStream_t stream) {
+                                         float out_scale, float cap, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (d <= 0 || d > AS_MAX_D || vd <= 0 || vd > AS_MAX_D || G <= 0 || H % G != 0 || page_size <= 0)
     return QD_ERR_UNSUPPORTED;
   const long long items = (long long)n_tokens * H;
   const unsigned blocks = (unsigned)((items + AS_WARPS - 1) / AS_WARPS);
   const size_t smem = (size_t)AS_WARPS * d * sizeof(float);
-  const AttnExtra ex = {chunk, gate, gate_ld, gate && gate_elem, out_scale, out_stride};
+  const AttnExtra ex = {chunk, gate, gate_ld, gate && gate_elem, out_scale, out_stride, cap};
   if (dtype == QD_F32)
     qd_launch(sink_attention_generic_kernel<float>, dim3(blocks), dim3(AS_WARPS * 32), smem, stream, (const float*)q,
               q_stride, (float*)out, out_stride, (const float*)kv, block_table, max_blocks, token_req, positions,
@@ -418,15 +431,36 @@ sink_attention_mma_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, co
 #pragma unroll
       for (int n = 0; n < TS_KEYS / 8; n++) ts_mma(s[n], qa[ks + 1], kb[n][2], kb[n][3]);
     }
+    float to_log2 = scale_log2;
+    if (ex.cap > 0.f) {
+      const float in = scale_log2 * 0.69314718055994531f / ex.cap;
+      float most = 0.f;
+#pragma unroll
+      for (int n = 0; n < TS_KEYS / 8; n++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) { s[n][i] *= in; most = fmaxf(most, fabsf(s[n][i])); }
+      if (__all_sync(0xffffffffu, most <= 0.25f)) {
+#pragma unroll
+        for (int n = 0; n < TS_KEYS / 8; n++)
+#pragma unroll
+          for (int i = 0; i < 4; i++) s[n][i] = as_tanh_small(s[n][i]);
+      } else {
+#pragma unroll
+        for (int n = 0; n < TS_KEYS / 8; n++)
+#pragma unroll
+          for (int i = 0; i < 4; i++) s[n][i] = fabsf(s[n][i]) <= 0.25f ? as_tanh_small(s[n][i]) : as_tanh_any(s[n][i]);
+      }
+      to_log2 = ex.cap * 1.4426950408889634f;
+    }
     // mask, scale (scores in units of log 2), row maxima
     float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
     for (int n = 0; n < TS_KEYS / 8; n++) {
       const int k0 = kt * TS_KEYS + n * 8 + 2 * tq, k1 = k0 + 1;
-      s[n][0] = (live0 && k0 <= p0 && k0 >= lo0) ? s[n][0] * scale_log2 : -INFINITY;
-      s[n][1] = (live0 && k1 <= p0 && k1 >= lo0) ? s[n][1] * scale_log2 : -INFINITY;
-      s[n][2] = (live1 && k0 <= p1 && k0 >= lo1) ? s[n][2] * scale_log2 : -INFINITY;
-      s[n][3] = (live1 && k1 <= p1 && k1 >= lo1) ? s[n][3] * scale_log2 : -INFINITY;
+      s[n][0] = (live0 && k0 <= p0 && k0 >= lo0) ? s[n][0] * to_log2 : -INFINITY;
+      s[n][1] = (live0 && k1 <= p0 && k1 >= lo0) ? s[n][1] * to_log2 : -INFINITY;
+      s[n][2] = (live1 && k0 <= p1 && k0 >= lo1) ? s[n][2] * to_log2 : -INFINITY;
+      s[n][3] = (live1 && k1 <= p1 && k1 >= lo1) ? s[n][3] * to_log2 : -INFINITY;
       mx0 = fmaxf(mx0, fmaxf(s[n][0], s[n][1]));
       mx1 = fmaxf(mx1, fmaxf(s[n][2], s[n][3]));
     }
@@ -614,13 +648,13 @@ extern "C" int qd_sink_attention_mma(const void* q, void* out, const void* kv, c
                                      int H, int G, int d, int vd, int page_size, float scale, int window,
                                      const float* sinks, int splits, float* part_o, float* part_ml,
                                      unsigned* tickets, int chunk, const float* gate, long long gate_ld,
-                                     int gate_elem, float out_scale, long long out_stride, cudaStream_t stream) {
+                                     int gate_elem, float out_scale, long long out_stride, float cap, cudaStream_t stream) {
   if (n_tokens <= 0 || n_requests <= 0) return 0;
   if (G <= 0 || H % G || H / G > TS_ROWS || d <= 0 || vd <= 0 || d > 128 || vd > 128 || d % 8 || vd % 8 ||
       page_size <= 0 || splits < 1 || splits > 64 || G > 65535 || (splits > 1 && (!part_o || !part_ml)) ||
       out_stride < (long long)H * vd || (out_stride & 1))
     return QD_ERR_UNSUPPORTED;
-  const AttnExtra ex = {chunk, gate, gate_ld, gate && gate_elem, out_scale, out_stride};
+  const AttnExtra ex = {chunk, gate, gate_ld, gate && gate_elem, out_scale, out_stride, cap};
   const float scale_log2 = scale * 1.4426950408889634f;
   int page_shift = -1;
   if ((page_size & (page_size - 1)) == 0)

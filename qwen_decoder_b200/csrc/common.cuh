@@ -34,6 +34,15 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// Gated activations, by code: silu(g) * u, or gelu(g) * u with gelu(z) = 0.5 z (1 + tanh(c (z + 0.044715 z^3))), c =
+// sqrt(2 / pi).  Since (1 + tanh(y)) / 2 = 1 / (1 + exp(-2 y)), both are g / (1 + exp(-a)) * u with another a.
+#define QD_ACT_SILU 0
+#define QD_ACT_GELU_TANH 2
+__device__ __forceinline__ float qd_gate_arg(float g, int act) {
+  return act == QD_ACT_GELU_TANH ? 1.5957691216057308f * fmaf(0.044715f * g * g, g, g) : g;
+}
+__device__ __forceinline__ float qd_gated(float g, float u, int act) { return g / (1.0f + expf(-qd_gate_arg(g, act))) * u; }
+
 // Sum over a block of up to 1024 threads; the order of additions depends only on
 // the block size, so a row's result does not depend on what else is in the batch.
 __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 33 floats */) {

@@ -548,7 +548,7 @@ extern "C" int qd_rope_kv_write_partial(const float* part, int n_parts, const fl
 // gate_up row = [ gate (F) | up (F) ];  out = gate / (1 + exp(-gate)) * up, in float32
 // (the reference's swiglu_kernel, gpu_kernels.cu:157-158).
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int F, size_t n) {
+__global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out, int F, size_t n, int act) {
   // no early start for the successor: it is a library product (the down projection), which gains nothing from it
   pdl_wait();
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -557,13 +557,13 @@ __global__ void swiglu_kernel(const T* __restrict__ gate_up, T* __restrict__ out
   int f = (int)(i - t * F);
   float g = to_float(gate_up[t * 2 * F + f]);
   float u = to_float(gate_up[t * 2 * F + F + f]);
-  out[i] = from_float<T>(g / (1.0f + expf(-g)) * u);
+  out[i] = from_float<T>(qd_gated(g, u, act));
 }
 
 // Eight features per thread and step with 16-byte loads and stores (bfloat16, F a multiple of 8); a thread
 // takes two steps, a grid apart, with all four loads in flight together.  The sigmoid uses the fast
 // exponential and division: their error (2^-21 relative) is far below the rounding of the bfloat16 result.
-__device__ __forceinline__ uint4 swiglu8(const uint4& g, const uint4& u) {
+__device__ __forceinline__ uint4 swiglu8(const uint4& g, const uint4& u, int act) {
   const __nv_bfloat162* gp = reinterpret_cast<const __nv_bfloat162*>(&g);
   const __nv_bfloat162* up = reinterpret_cast<const __nv_bfloat162*>(&u);
   uint4 o;
@@ -571,13 +571,14 @@ __device__ __forceinline__ uint4 swiglu8(const uint4& g, const uint4& u) {
 #pragma unroll
   for (int k = 0; k < 4; k++) {
     float2 gf = __bfloat1622float2(gp[k]), uf = __bfloat1622float2(up[k]);
-    op[k] = __floats2bfloat162_rn(__fdividef(gf.x, 1.0f + __expf(-gf.x)) * uf.x,
-                                  __fdividef(gf.y, 1.0f + __expf(-gf.y)) * uf.y);
+    op[k] = __floats2bfloat162_rn(__fdividef(gf.x, 1.0f + __expf(-fmaxf(qd_gate_arg(gf.x, act), -80.0f))) * uf.x,
+                                  __fdividef(gf.y, 1.0f + __expf(-fmaxf(qd_gate_arg(gf.y, act), -80.0f))) * uf.y);
   }
   return o;
 }
 
-__global__ void swiglu_vec_kernel(const bf16* __restrict__ gate_up, bf16* __restrict__ out, int F8, size_t n8) {
+__global__ void swiglu_vec_kernel(const bf16* __restrict__ gate_up, bf16* __restrict__ out, int F8, size_t n8,
+                                  int act) {
   pdl_wait();        // as above: the successor is a library product
   const size_t half = (n8 + 1) / 2;
   const size_t i0 = (size_t)blockIdx.x * blockDim.x + threadIdx.x, i1 = i0 + half;
@@ -589,15 +590,15 @@ __global__ void swiglu_vec_kernel(const bf16* __restrict__ gate_up, bf16* __rest
   uint4 g0 = base[t0 * 2 * F8 + a0], u0 = base[t0 * 2 * F8 + F8 + a0];
   uint4 g1 = make_uint4(0, 0, 0, 0), u1 = g1;
   if (two) { g1 = base[t1 * 2 * F8 + a1]; u1 = base[t1 * 2 * F8 + F8 + a1]; }
-  reinterpret_cast<uint4*>(out)[i0] = swiglu8(g0, u0);
-  if (two) reinterpret_cast<uint4*>(out)[i1] = swiglu8(g1, u1);
+  reinterpret_cast<uint4*>(out)[i0] = swiglu8(g0, u0, act);
+  if (two) reinterpret_cast<uint4*>(out)[i1] = swiglu8(g1, u1, act);
 }
 
 // The same from the float32 partial sums of a split-K product: part [n_parts, T, 2F]; the shares are added
 // first, exactly (float32), and the result is rounded to bfloat16 once.  Four features per thread with 16-byte
 // loads, all shares of a thread's gate and up values asked for before any is used (in groups of four shares).
 __global__ void swiglu_partial_kernel(const float* __restrict__ part, int n_parts, const float* __restrict__ bias,
-                                      bf16* __restrict__ out, int F4, size_t n4, size_t part_stride4) {
+                                      bf16* __restrict__ out, int F4, size_t n4, size_t part_stride4, int act) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -621,8 +622,8 @@ __global__ void swiglu_partial_kernel(const float* __restrict__ part, int n_part
       u.x += uv[q].x; u.y += uv[q].y; u.z += uv[q].z; u.w += uv[q].w;
     }
   }
-  __nv_bfloat162 o0 = __floats2bfloat162_rn(g.x / (1.0f + expf(-g.x)) * u.x, g.y / (1.0f + expf(-g.y)) * u.y);
-  __nv_bfloat162 o1 = __floats2bfloat162_rn(g.z / (1.0f + expf(-g.z)) * u.z, g.w / (1.0f + expf(-g.w)) * u.w);
+  __nv_bfloat162 o0 = __floats2bfloat162_rn(qd_gated(g.x, u.x, act), qd_gated(g.y, u.y, act));
+  __nv_bfloat162 o1 = __floats2bfloat162_rn(qd_gated(g.z, u.z, act), qd_gated(g.w, u.w, act));
   uint2 o;
   o.x = *reinterpret_cast<unsigned*>(&o0);
   o.y = *reinterpret_cast<unsigned*>(&o1);
@@ -632,31 +633,36 @@ __global__ void swiglu_partial_kernel(const float* __restrict__ part, int n_part
 // out [T, F] bfloat16 = silu(bias[f] + sum_p part[p, t, f]) * (bias[F + f] + sum_p part[p, t, F + f]); bias [2F] or null;
 // F a multiple of 4, 16-byte aligned.
 extern "C" int qd_swiglu_partial(const float* part, int n_parts, const float* bias, void* out, int T, int F,
-                                 cudaStream_t stream) {
+                                 int act, cudaStream_t stream) {
   if (T <= 0 || F <= 0) return 0;
   if (n_parts < 1 || F % 4 != 0 || (((uintptr_t)part | (uintptr_t)bias) & 15) || (((uintptr_t)out) & 7))
     return QD_ERR_UNSUPPORTED;
   const size_t n4 = (size_t)T * F / 4;
   qd_launch(swiglu_partial_kernel, dim3((unsigned)((n4 + 127) / 128)), dim3(128), 0, stream, part, n_parts, bias, (bf16*)out,
-            F / 4, n4, (size_t)T * 2 * F / 4);
+            F / 4, n4, (size_t)T * 2 * F / 4, act);
   return qd_last_error();
 }
 
-extern "C" int qd_swiglu(const void* gate_up, void* out, int dtype, int T, int F, cudaStream_t stream) {
+// out[t, f] = act(gate_up[t, f]) * gate_up[t, F + f]; ``act``: QD_ACT_*.
+extern "C" int qd_gate_mul(const void* gate_up, void* out, int dtype, int T, int F, int act, cudaStream_t stream) {
   size_t n = (size_t)T * F;
   if (n == 0) return 0;
   if (dtype == QD_BF16 && F % 8 == 0 && !(((uintptr_t)gate_up | (uintptr_t)out) & 15)) {
     size_t n8 = n / 8;
     qd_launch(swiglu_vec_kernel, dim3((unsigned)(((n8 + 1) / 2 + 255) / 256)), dim3(256), 0, stream, (const bf16*)gate_up,
-              (bf16*)out, F / 8, n8);
+              (bf16*)out, F / 8, n8, act);
     return qd_last_error();
   }
   unsigned blocks = (unsigned)((n + 255) / 256);
   if (dtype == QD_F32)
-    qd_launch(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, F, n);
+    qd_launch(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gate_up, (float*)out, F, n, act);
   else if (dtype == QD_BF16)
-    qd_launch(swiglu_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, F, n);
+    qd_launch(swiglu_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gate_up, (bf16*)out, F, n, act);
   else
     return QD_ERR_UNSUPPORTED;
   return qd_last_error();
+}
+
+extern "C" int qd_swiglu(const void* gate_up, void* out, int dtype, int T, int F, cudaStream_t stream) {
+  return qd_gate_mul(gate_up, out, dtype, T, F, QD_ACT_SILU, stream);
 }

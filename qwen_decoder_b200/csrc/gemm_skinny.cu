@@ -43,7 +43,7 @@ template <int TN, int EPI, typename TO>
 __global__ void __launch_bounds__(SK_WARPS * 32)
 gemm_skinny_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, long long ldx,
                    const float* __restrict__ bias, TO* __restrict__ out, long long ldo,
-                   float* __restrict__ part, int T, int N, int K, int splits) {
+                   float* __restrict__ part, int T, int N, int K, int splits, int act) {
   __shared__ float red[SK_WARPS][16][TN * 8 + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int j = lane & 3, r = lane >> 2;
@@ -135,7 +135,7 @@ gemm_skinny_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, long 
 #pragma unroll
       for (int w = 0; w < SK_WARPS; w++) { gate += red[w][row][tok]; up += red[w][row + 8][tok]; }
       if (bias) { gate += bias[f]; up += bias[F + f]; }
-      out[(size_t)tok * ldo + f] = from_float<TO>(gate / (1.0f + expf(-gate)) * up);
+      out[(size_t)tok * ldo + f] = from_float<TO>(qd_gated(gate, up, act));
     }
   } else {
     for (int idx = threadIdx.x; idx < 16 * TN * 8; idx += SK_WARPS * 32) {
@@ -158,25 +158,25 @@ gemm_skinny_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, long 
 template <int TN>
 static int launch_skinny(const bf16* W, const bf16* X, long long ldx, const float* bias, void* out,
                          int out_dtype, long long ldo, float* part, int T, int N, int K, int splits, int epi,
-                         cudaStream_t stream) {
+                         int act, cudaStream_t stream) {
   dim3 block(SK_WARPS * 32);
   if (epi == EPI_SWIGLU) {
     dim3 grid((N / 2 + 7) / 8, 1);
     if (out_dtype != QD_BF16) return QD_ERR_UNSUPPORTED;
     qd_launch(gemm_skinny_kernel<TN, EPI_SWIGLU, bf16>, dim3(grid), dim3(block), 0, stream, W, X, ldx, bias, (bf16*)out, ldo,
-                                                                         nullptr, T, N, K, 1);
+                                                                         nullptr, T, N, K, 1, act);
   } else if (epi == EPI_PARTIAL) {
     dim3 grid((N + 15) / 16, splits);
     qd_launch(gemm_skinny_kernel<TN, EPI_PARTIAL, float>, dim3(grid), dim3(block), 0, stream, W, X, ldx, nullptr, nullptr, 0, part,
-                                                                           T, N, K, splits);
+                                                                           T, N, K, splits, act);
   } else {
     dim3 grid((N + 15) / 16, 1);
     if (out_dtype == QD_BF16)
       qd_launch(gemm_skinny_kernel<TN, EPI_STORE, bf16>, dim3(grid), dim3(block), 0, stream, W, X, ldx, bias, (bf16*)out, ldo,
-                                                                          nullptr, T, N, K, 1);
+                                                                          nullptr, T, N, K, 1, act);
     else if (out_dtype == QD_F32)
       qd_launch(gemm_skinny_kernel<TN, EPI_STORE, float>, dim3(grid), dim3(block), 0, stream, W, X, ldx, bias, (float*)out, ldo,
-                                                                           nullptr, T, N, K, 1);
+                                                                           nullptr, T, N, K, 1, act);
     else
       return QD_ERR_UNSUPPORTED;
   }
@@ -185,20 +185,23 @@ static int launch_skinny(const bf16* W, const bf16* X, long long ldx, const floa
 
 // epi 0: out[T, N] = X W^T + bias (out_dtype bf16 or f32).  epi 1: part[splits, T, N] float32 partial
 // sums over ``splits`` shares of K (no bias).  epi 2: W is [2F, K] = gate rows then up rows, N = 2F,
-// out[T, F] = silu(X Wg^T + bias_g) * (X Wu^T + bias_u), bfloat16 (bias [2F] or null).  X rows are ldx elements apart, out rows ldo.
+// out[T, F] = silu(X Wg^T + bias_g) * (X Wu^T + bias_u), bfloat16 (bias [2F] or null);
+// epi + 256 * act: another activation in silu's place (QD_ACT_*).  X rows are ldx elements apart, out rows ldo.
 extern "C" int qd_gemm_skinny(const void* W, const void* X, long long ldx, const float* bias, void* out,
                               int out_dtype, long long ldo, float* part, int T, int N, int K, int splits,
                               int epi, cudaStream_t stream) {
   if (T <= 0 || N <= 0) return 0;
   if (T > 64 || K <= 0 || K % 8 != 0 || ldx % 8 != 0 || splits < 1 || splits > 65535) return QD_ERR_UNSUPPORTED;
   if (((uintptr_t)W & 15) || ((uintptr_t)X & 15)) return QD_ERR_UNSUPPORTED;
+  const int act = epi >> 8;
+  epi &= 255;
   if (epi == EPI_SWIGLU && (N & 1)) return QD_ERR_UNSUPPORTED;
   if (epi == EPI_PARTIAL && !part) return QD_ERR_UNSUPPORTED;
   if (epi != EPI_PARTIAL && splits != 1) return QD_ERR_UNSUPPORTED;
   const bf16* w = (const bf16*)W;
   const bf16* x = (const bf16*)X;
-  if (T <= 8) return launch_skinny<1>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, stream);
-  if (T <= 16) return launch_skinny<2>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, stream);
-  if (T <= 32) return launch_skinny<4>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, stream);
-  return launch_skinny<8>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, stream);
+  if (T <= 8) return launch_skinny<1>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, act, stream);
+  if (T <= 16) return launch_skinny<2>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, act, stream);
+  if (T <= 32) return launch_skinny<4>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, act, stream);
+  return launch_skinny<8>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, act, stream);
 }

@@ -71,7 +71,7 @@ __global__ void __launch_bounds__(ST_THREADS)
 gemm_stream_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, long long ldx,
                    const float* __restrict__ bias, TO* __restrict__ out, long long ldo,
                    float* __restrict__ part, int T, int N, int K, int splits, int n_tiles,
-                   int* __restrict__ status) {
+                   int* __restrict__ status, int act) {
   constexpr int NST = StageCfg<TN>::STAGES;
   constexpr int STAGE_BYTES = StageCfg<TN>::BYTES;
   extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -245,7 +245,7 @@ gemm_stream_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, long 
           up += red[((size_t)w * 16 + row + 8) * RED_LD + tok];
         }
         if (bias) { gate += bias[f]; up += bias[F + f]; }
-        out[(size_t)tok * ldo + f] = from_float<TO>(gate / (1.0f + expf(-gate)) * up);
+        out[(size_t)tok * ldo + f] = from_float<TO>(qd_gated(gate, up, act));
       }
     } else {
       for (int idx = threadIdx.x; idx < 16 * TN * 8; idx += ST_CONSUMERS * 32) {
@@ -357,7 +357,7 @@ __global__ void __launch_bounds__(ST_THREADS, 2)
 gemm_stream_xres_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, long long ldx,
                         const float* __restrict__ bias, TO* __restrict__ out, long long ldo,
                         float* __restrict__ part, int T, int N, int K, int splits, int n_tiles,
-                        int* __restrict__ status) {
+                        int* __restrict__ status, int act) {
   constexpr int NST = XR_STAGES;
   extern __shared__ __align__(128) unsigned char smem_raw[];
   unsigned char* stages = smem_raw;                                               // NST x 16 rows of W
@@ -474,7 +474,7 @@ gemm_stream_xres_kernel(const bf16* __restrict__ W, const bf16* __restrict__ X, 
           up += red[((size_t)w * 16 + row + 8) * RED_LD + tok];
         }
         if (bias) { gate += bias[f]; up += bias[F + f]; }
-        out[(size_t)tok * ldo + f] = from_float<TO>(gate / (1.0f + expf(-gate)) * up);
+        out[(size_t)tok * ldo + f] = from_float<TO>(qd_gated(gate, up, act));
       }
     } else {
       for (int idx = threadIdx.x; idx < 16 * TN * 8; idx += ST_CONSUMERS * 32) {
@@ -510,7 +510,7 @@ struct FfnArgs {
   const float* b1;                                                              // [2F] added before SwiGLU, or null
   bf16* h; long long ldh;                                                       // [T, F]
   const bf16* w2; int N2, K2, n_tiles2, splits2; float* part;                   // [D, F] -> [splits2, T, D]
-  int T;
+  int T, act;                                                                   // act: QD_ACT_*
   unsigned* gbar;            // FFN_SYNC_WORDS words, zero before first use: per chunk of ST_KC columns of h the
                              // row tiles of the first product that are written; last word: CTAs past their wait
   int* status;
@@ -713,7 +713,7 @@ ffn_stream_kernel(const FfnArgs a) {
         up += red[((size_t)w * 16 + row + 8) * RED_LD + tok];
       }
       if (a.b1) { gate += a.b1[f]; up += a.b1[F + f]; }
-      a.h[(size_t)tok * a.ldh + f] = __float2bfloat16_rn(gate / (1.0f + expf(-gate)) * up);
+      a.h[(size_t)tok * a.ldh + f] = __float2bfloat16_rn(qd_gated(gate, up, a.act));
     }
     asm volatile("bar.sync 1, %0;" ::"n"(ST_CONSUMERS * 32) : "memory");
     // this tile's 8 columns of h are written (by the threads that met at the barrier above): the telling warp
@@ -779,7 +779,7 @@ static bool xres_fits(int T, int K, int splits, int max_ctas) {
 template <int TN>
 static int launch_stream_xres(const bf16* W, const bf16* X, long long ldx, const float* bias, void* out, int out_dtype,
                               long long ldo, float* part, int T, int N, int K, int splits, int epi, int max_ctas,
-                              cudaStream_t stream) {
+                              int act, cudaStream_t stream) {
   int* status = status_word();
   if (!status) return QD_ERR_UNSUPPORTED;
   int n_tiles = epi == EPI_SWIGLU ? (N / 2 + 7) / 8 : (N + 15) / 16;
@@ -793,7 +793,7 @@ static int launch_stream_xres(const bf16* W, const bf16* X, long long ldx, const
   do {                                                                                                           \
     cudaFuncSetAttribute(gemm_stream_xres_kernel<TN, E, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     qd_launch(gemm_stream_xres_kernel<TN, E, TO>, dim3(grid), dim3(ST_THREADS), smem, stream, W, X, ldx, bias,       \
-              (TO*)out, ldo, part, T, N, K, splits, n_tiles, status);                                            \
+              (TO*)out, ldo, part, T, N, K, splits, n_tiles, status, act);                                            \
   } while (0)
   if (epi == EPI_SWIGLU) {
     if (out_dtype != QD_BF16) return QD_ERR_UNSUPPORTED;
@@ -814,7 +814,7 @@ static int launch_stream_xres(const bf16* W, const bf16* X, long long ldx, const
 template <int TN>
 static int launch_stream(const bf16* W, const bf16* X, long long ldx, const float* bias, void* out, int out_dtype,
                          long long ldo, float* part, int T, int N, int K, int splits, int epi, int max_ctas,
-                         cudaStream_t stream) {
+                         int act, cudaStream_t stream) {
   int* status = status_word();
   if (!status) return QD_ERR_UNSUPPORTED;
   int n_tiles = epi == EPI_SWIGLU ? (N / 2 + 7) / 8 : (N + 15) / 16;
@@ -825,7 +825,7 @@ static int launch_stream(const bf16* W, const bf16* X, long long ldx, const floa
   do {                                                                                                      \
     cudaFuncSetAttribute(gemm_stream_kernel<TN, E, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     qd_launch(gemm_stream_kernel<TN, E, TO>, dim3(grid), dim3(ST_THREADS), smem, stream, W, X, ldx, bias,   \
-              (TO*)out, ldo, part, T, N, K, splits, n_tiles, status);                                       \
+              (TO*)out, ldo, part, T, N, K, splits, n_tiles, status, act);                                       \
   } while (0)
   if (epi == EPI_SWIGLU) {
     if (out_dtype != QD_BF16) return QD_ERR_UNSUPPORTED;
@@ -852,27 +852,29 @@ extern "C" int qd_gemm_stream(const void* W, const void* X, long long ldx, const
   if (T > 64 || K <= 0 || K % 8 != 0 || ldx % 8 != 0 || splits < 1 || max_ctas < 1) return QD_ERR_UNSUPPORTED;
   if (splits > (K + ST_KC - 1) / ST_KC) return QD_ERR_UNSUPPORTED;
   if (((uintptr_t)W & 15) || ((uintptr_t)X & 15)) return QD_ERR_UNSUPPORTED;
+  const int act = epi >> 8;                                 // the gated epilogue's activation (QD_ACT_*)
+  epi &= 255;
   if (epi == EPI_SWIGLU && (N & 1)) return QD_ERR_UNSUPPORTED;
   if (epi == EPI_PARTIAL && !part) return QD_ERR_UNSUPPORTED;
   if (epi != EPI_PARTIAL && splits != 1) return QD_ERR_UNSUPPORTED;
   const bf16* w = (const bf16*)W;
   const bf16* x = (const bf16*)X;
   if (xres_fits(T, K, splits, max_ctas))
-    return T <= 8 ? launch_stream_xres<1>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, stream)
-                  : launch_stream_xres<2>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, stream);
-  if (T <= 8) return launch_stream<1>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, stream);
-  if (T <= 16) return launch_stream<2>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, stream);
-  if (T <= 32) return launch_stream<4>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, stream);
-  return launch_stream<8>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, stream);
+    return T <= 8 ? launch_stream_xres<1>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, act, stream)
+                  : launch_stream_xres<2>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, act, stream);
+  if (T <= 8) return launch_stream<1>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, act, stream);
+  if (T <= 16) return launch_stream<2>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, act, stream);
+  if (T <= 32) return launch_stream<4>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, act, stream);
+  return launch_stream<8>(w, x, ldx, bias, out, out_dtype, ldo, part, T, N, K, splits, epi, max_ctas, act, stream);
 }
 
-// The feed-forward of up to 8 tokens in one launch: h = silu(x Wg^T) * (x Wu^T) (w1 = [Wg; Wu], [2F, D]) and
+// The feed-forward of up to 8 tokens in one launch: h = act(x Wg^T) * (x Wu^T) (``act``: QD_ACT_*; w1 = [Wg; Wu], [2F, D]) and
 // part[s] = partial sums of h W2^T over `splits2` shares of F; `b1` [2F] (or null) is added to gate and up.  `gbar`: 64 zeroed words of device memory that
 // stay with the caller (the kernel leaves them zero for the next launch).  Refuses what it cannot take
 // (more than 8 tokens, D above 2,048, a share of F wider than 2,048, more CTAs than fit on the device at once).
 extern "C" int qd_ffn_stream(const void* w1, const float* b1, const void* x, long long ldx, void* h, long long ldh,
                              const void* w2, float* part, int T, int D, int F, int splits2, unsigned* gbar, int max_ctas,
-                             long long* timeline, cudaStream_t stream) {
+                             int act, long long* timeline, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (T > 8 || D <= 0 || F <= 0 || D % 8 != 0 || F % 8 != 0 || ldx % 8 != 0 || ldh % 8 != 0 || D > XR_KMAX ||
       splits2 < 1 || !gbar || !part || (F + ST_KC - 1) / ST_KC > FFN_SYNC_WORDS - 1)
@@ -898,7 +900,7 @@ extern "C" int qd_ffn_stream(const void* w1, const float* b1, const void* x, lon
   a.w1 = (const bf16*)w1; a.b1 = b1; a.x1 = (const bf16*)x; a.ldx1 = ldx; a.N1 = 2 * F; a.K1 = D; a.n_tiles1 = (F + 7) / 8;
   a.h = (bf16*)h; a.ldh = ldh;
   a.w2 = (const bf16*)w2; a.N2 = D; a.K2 = F; a.n_tiles2 = (D + 15) / 16; a.splits2 = splits2; a.part = part;
-  a.T = T; a.gbar = gbar; a.status = status; a.timeline = timeline;
+  a.T = T; a.act = act; a.gbar = gbar; a.status = status; a.timeline = timeline;
   int grid = per_sm * sms;
   if (grid > max_ctas) grid = max_ctas;
   if (grid > a.n_tiles1) grid = a.n_tiles1;

@@ -97,6 +97,7 @@ __device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence:
 __device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
 
 struct TcParams {
+  int act;                // the gated epilogue's activation (QD_ACT_*)
   int T, N, K;            // tokens, output features (for SwiGLU: 2F rows of W), contraction
   int BN;                 // tokens per tile: 16, 32, 64, 128 or 256
   int splits;             // shares of K (partial sums) or 1
@@ -295,7 +296,7 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
               float a = v[i];
               if (EPI == EPI_SWIGLU) {
                 a += bv;
-                out[(size_t)tok * p.ldo + feature] = from_float<TO>(a / (1.0f + expf(-a)) * (u[i] + bu));
+                out[(size_t)tok * p.ldo + feature] = from_float<TO>(qd_gated(a, u[i] + bu, p.act));
               } else if (EPI == EPI_PARTIAL) {
                 part[((size_t)sp * p.T + tok) * p.N + feature] = a;
               } else {
@@ -375,6 +376,8 @@ extern "C" int qd_gemm_tc5(const void* W, const void* X, long long ldx, const fl
   if (T <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8 != 0 || ldx % 8 != 0 || splits < 1 || max_ctas < 1) return QD_ERR_UNSUPPORTED;
   if (((uintptr_t)W & 15) || ((uintptr_t)X & 15)) return QD_ERR_UNSUPPORTED;
+  const int act = epi >> 8;                                // epi + 256 * act: another activation in silu's place
+  epi &= 255;
   if (epi == EPI_SWIGLU && (N & 1)) return QD_ERR_UNSUPPORTED;
   if (epi == EPI_PARTIAL && !part) return QD_ERR_UNSUPPORTED;
   if (epi != EPI_PARTIAL && splits != 1) return QD_ERR_UNSUPPORTED;
@@ -384,7 +387,7 @@ extern "C" int qd_gemm_tc5(const void* W, const void* X, long long ldx, const fl
   if (!status) return QD_ERR_UNSUPPORTED;
 
   TcParams p;
-  p.T = T; p.N = N; p.K = K; p.splits = splits; p.ldo = ldo;
+  p.act = act; p.T = T; p.N = N; p.K = K; p.splits = splits; p.ldo = ldo;
   p.BN = T <= 16 ? 16 : T <= 32 ? 32 : T <= 64 ? 64 : T <= 128 ? 128 : 256;
   if (epi == EPI_SWIGLU && p.BN > 128) p.BN = 128;       // two accumulators x two buffers must fit 512 columns
   const int feats = epi == EPI_SWIGLU ? N / 2 : N;

@@ -2,7 +2,7 @@
 //
 //   y = sum of the branch output's partial sums (+ a bias per channel)
 //   x[s] += G(y; post_w, post_eps, post_groups)          (without post_w: x[s] += y)
-//   out[r] = G(x[s]; pre_w, pre_eps, pre_groups)          (without pre_w: nothing is written), s = rows[r] (or r)
+//   out[r] = G(x[s]; pre_w, pre_eps, pre_groups), s = rows[r] (or r);  without pre_w out[r] = x[s], and without out nothing is written
 //
 // G(v; w, eps, n): v is cut into n equal consecutive parts, every part is divided by its own sqrt(mean(part^2) + eps),
 // and the whole is multiplied by w.  float32 throughout; one CTA per row; the order of a part's sum depends on the
@@ -141,7 +141,15 @@ group_add_norm_warp_kernel(GroupNorm a) {
       if (lane == 0 && i < n4) sums[i >> 5] = t;
     }
   }
-  if (!a.pre_w) return;
+  if (!a.out) return;
+  if (!a.pre_w) {                                     // the sum itself, rounded
+#pragma unroll
+    for (int q = 0; q < VPT; q++) {
+      const int i = threadIdx.x + q * blockDim.x;
+      if (i < n4) out4(a, (size_t)r, i, xv[q]);
+    }
+    return;
+  }
   __syncthreads();
   const int part4 = n4 / a.pre_groups;
 #pragma unroll
@@ -205,7 +213,15 @@ group_add_norm_vec_kernel(GroupNorm a) {
     }
     if (a.pre_w) sq[i] = sq4(xv[q]);
   }
-  if (!a.pre_w) return;
+  if (!a.out) return;
+  if (!a.pre_w) {
+#pragma unroll
+    for (int q = 0; q < VPT; q++) {
+      const int i = threadIdx.x + q * blockDim.x;
+      if (i < n4) out4(a, (size_t)r, i, xv[q]);
+    }
+    return;
+  }
   group_factors(sq, n4, a.pre_groups, pre_part4 * 4, a.pre_eps, scratch, f);
 #pragma unroll
   for (int q = 0; q < VPT; q++) {
@@ -253,10 +269,10 @@ group_add_norm_kernel(GroupNorm a) {
     v[i] = x;
     sq[i] = x * x;
   }
-  if (!a.pre_w) return;
-  group_factors(sq, D, a.pre_groups, pre_part, a.pre_eps, scratch, f);
+  if (!a.out) return;
+  if (a.pre_w) group_factors(sq, D, a.pre_groups, pre_part, a.pre_eps, scratch, f);
   for (int i = threadIdx.x; i < D; i += blockDim.x) {
-    const float o = v[i] * f[i / pre_part] * a.pre_w[i];
+    const float o = a.pre_w ? v[i] * f[i / pre_part] * a.pre_w[i] : v[i];
     if (a.out_dtype == QD_F32) reinterpret_cast<float*>(a.out)[(size_t)r * D + i] = o;
     else reinterpret_cast<bf16*>(a.out)[(size_t)r * D + i] = __float2bfloat16_rn(o);
   }
@@ -273,7 +289,7 @@ extern "C" int qd_group_add_norm(float* x, const void* delta, int delta_dtype, i
   if (!pre_w) pre_groups = 1;
   if (D <= 0 || post_groups < 1 || pre_groups < 1 || D % post_groups || D % pre_groups || n_parts < 1 || (pre_w && !out) ||
       (delta && delta_dtype != QD_F32 && (delta_dtype != QD_BF16 || n_parts != 1)) ||
-      (pre_w && out_dtype != QD_F32 && out_dtype != QD_BF16))
+      (out && out_dtype != QD_F32 && out_dtype != QD_BF16))
     return QD_ERR_UNSUPPORTED;
   const GroupNorm a = {x, delta, delta_dtype, n_parts, (size_t)part_stride, delta_bias, post_w, post_eps, post_groups,
                        pre_w, pre_eps, pre_groups, out, out_dtype, rows, D, write_back};

@@ -6,6 +6,7 @@
 // themselves -- every head of a token reads the same rows, so a CTA stages a tile of rows once for
 // all its heads -- and the result is carried out of the latent space afterwards (``expand``).
 //
+//   (the rotated parts turn by the token's position in adjacent or in half-split pairs)
 //   prep     RMS norms of the query latent and of c (float32), rotation of kr, write of the cache row
 //   absorb   qcat[t, h] = [ Wuk_h^T qn[t, h] | rotate(qr[t, h]) ]                    float32
 //   attend   o_lat[t, h] = softmax_j<=pos(qcat[t, h] . row_j * scale) c_j            float32, paged, split over keys
@@ -32,6 +33,17 @@ template <> struct Vec16<bf16> {
   }
 };
 
+// Element e of a rotated part whose first 2 * half elements turn: pairs (2p, 2p + 1), or with ``pairing`` 1
+// (p, p + half); cos_r and sin_r are the position's table rows.
+__device__ __forceinline__ float la_turn(const float* x, int e, int half, int pairing, const float* cos_r, const float* sin_r) {
+  if (e >= 2 * half) return x[e];
+  const int p = pairing ? (e < half ? e : e - half) : e >> 1;
+  const bool second = pairing ? e >= half : (e & 1);
+  const float a = x[pairing ? p : 2 * p], b = x[pairing ? p + half : 2 * p + 1];
+  const float c = cos_r[p], s = sin_r[p];
+  return second ? b * c + a * s : a * c - b * s;
+}
+
 #define LA_WARPS 8
 #define LA_TILE 32          // keys per staged tile
 #define LA_MAX_R 512        // latent size the attend kernel takes (16 accumulators a lane)
@@ -47,7 +59,7 @@ latent_prep_kernel(const float* __restrict__ u, long long ldu, int q_off, int q_
                    const float* __restrict__ wq_norm, const float* __restrict__ wkv_norm, float eps,
                    const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims,
                    const int* __restrict__ positions, const int* __restrict__ slot_map, TC* __restrict__ cq,
-                   TC* __restrict__ cache, int write_cache) {
+                   TC* __restrict__ cache, int write_cache, int pairing) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float scratch[40];
@@ -67,13 +79,8 @@ latent_prep_kernel(const float* __restrict__ u, long long ldu, int q_off, int q_
   for (int i = threadIdx.x; i < r; i += blockDim.x) dst[i] = from_float<TC>(row[kv_off + i] * ik * wkv_norm[i]);
   const int pos = positions[t];
   const int half = rot_dims >> 1;
-  for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    float c = cos_t[(size_t)pos * half + i], s = sin_t[(size_t)pos * half + i];
-    float a = row[kv_off + r + 2 * i], b = row[kv_off + r + 2 * i + 1];
-    dst[r + 2 * i] = from_float<TC>(a * c - b * s);
-    dst[r + 2 * i + 1] = from_float<TC>(b * c + a * s);
-  }
-  for (int i = rot_dims + threadIdx.x; i < dr; i += blockDim.x) dst[r + i] = from_float<TC>(row[kv_off + r + i]);
+  for (int i = threadIdx.x; i < dr; i += blockDim.x)
+    dst[r + i] = from_float<TC>(la_turn(row + kv_off + r, i, half, pairing, cos_t + (size_t)pos * half, sin_t + (size_t)pos * half));
 }
 
 // ----------------------------------------------------------------------------- absorb
@@ -83,7 +90,7 @@ __global__ void __launch_bounds__(256)
 latent_absorb_kernel(const float* __restrict__ q, long long ldq, const TW* __restrict__ wuk, float* __restrict__ qcat,
                      int T, int H, int dn, int dr, int r, const float* __restrict__ cos_t,
                      const float* __restrict__ sin_t, int rot_dims, const int* __restrict__ positions,
-                     const float* __restrict__ pre) {
+                     const float* __restrict__ pre, int pairing) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float qs[];                // [LA_TT][dn]
@@ -120,16 +127,8 @@ latent_absorb_kernel(const float* __restrict__ q, long long ldq, const TW* __res
   for (int i = threadIdx.x; i < nt * dr; i += blockDim.x) {
     int tt = i / dr, e = i - tt * dr;
     const float* qr = q + (size_t)(t0 + tt) * qw + (size_t)h * (dn + dr) + dn;
-    float v;
-    if (e < rot_dims) {
-      int pr = e >> 1, pos = positions[t0 + tt];
-      float c = cos_t[(size_t)pos * half + pr], s = sin_t[(size_t)pos * half + pr];
-      float a = qr[2 * pr], b = qr[2 * pr + 1];
-      v = (e & 1) ? b * c + a * s : a * c - b * s;
-    } else {
-      v = qr[e];
-    }
-    qcat[((size_t)(t0 + tt) * H + h) * W + r + e] = v;
+    const size_t at = (size_t)positions[t0 + tt] * half;
+    qcat[((size_t)(t0 + tt) * H + h) * W + r + e] = la_turn(qr, e, half, pairing, cos_t + at, sin_t + at);
   }
 }
 
@@ -141,7 +140,7 @@ __global__ void __launch_bounds__(256)
 latent_absorb_vec_kernel(const float* __restrict__ q, long long ldq, const TW* __restrict__ wuk,
                          float* __restrict__ qcat, int T, int H, int dn, int dr, int r,
                          const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims,
-                         const int* __restrict__ positions) {
+                         const int* __restrict__ positions, int pairing) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int V = Vec16<TW>::N;
@@ -194,16 +193,8 @@ latent_absorb_vec_kernel(const float* __restrict__ q, long long ldq, const TW* _
   for (int i = threadIdx.x; i < nt * dr; i += blockDim.x) {
     int tt = i / dr, e = i - tt * dr;
     const float* qr = q + (size_t)(t0 + tt) * qw + (size_t)h * (dn + dr) + dn;
-    float v;
-    if (e < rot_dims) {
-      int pr = e >> 1, pos = positions[t0 + tt];
-      float c = cos_t[(size_t)pos * half + pr], sn = sin_t[(size_t)pos * half + pr];
-      float a = qr[2 * pr], b = qr[2 * pr + 1];
-      v = (e & 1) ? b * c + a * sn : a * c - b * sn;
-    } else {
-      v = qr[e];
-    }
-    qcat[((size_t)(t0 + tt) * H + h) * W + r + e] = v;
+    const size_t at = (size_t)positions[t0 + tt] * half;
+    qcat[((size_t)(t0 + tt) * H + h) * W + r + e] = la_turn(qr, e, half, pairing, cos_t + at, sin_t + at);
   }
 }
 
@@ -617,15 +608,15 @@ static inline bool lm_enabled() {
 extern "C" int qd_latent_prep(const float* u, long long ldu, int q_off, int q_rank, int kv_off, int r, int dr,
                               const float* wq_norm, const float* wkv_norm, float eps, const float* cos_t,
                               const float* sin_t, int rot_dims, const int* positions, const int* slot_map, void* cq,
-                              void* cache, int dtype, int write_cache, int T, cudaStream_t stream) {
+                              void* cache, int dtype, int write_cache, int T, int pairing, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (rot_dims % 2 || rot_dims > dr || q_rank < 0 || r <= 0) return QD_ERR_UNSUPPORTED;
   if (dtype == QD_F32)
     qd_launch(latent_prep_kernel<float>, dim3(T), dim3(256), 0, stream, u, ldu, q_off, q_rank, kv_off, r, dr, wq_norm,
-              wkv_norm, eps, cos_t, sin_t, rot_dims, positions, slot_map, (float*)cq, (float*)cache, write_cache);
+              wkv_norm, eps, cos_t, sin_t, rot_dims, positions, slot_map, (float*)cq, (float*)cache, write_cache, pairing);
   else if (dtype == QD_BF16)
     qd_launch(latent_prep_kernel<bf16>, dim3(T), dim3(256), 0, stream, u, ldu, q_off, q_rank, kv_off, r, dr, wq_norm,
-              wkv_norm, eps, cos_t, sin_t, rot_dims, positions, slot_map, (bf16*)cq, (bf16*)cache, write_cache);
+              wkv_norm, eps, cos_t, sin_t, rot_dims, positions, slot_map, (bf16*)cq, (bf16*)cache, write_cache, pairing);
   else
     return QD_ERR_UNSUPPORTED;
   return qd_last_error();
@@ -635,7 +626,7 @@ extern "C" int qd_latent_prep(const float* u, long long ldu, int q_off, int q_ra
 // lays it beside the rotated part.
 extern "C" int qd_latent_absorb(const float* q, long long ldq, const void* wuk, int w_dtype, float* qcat, int T, int H, int dn, int dr,
                                 int r, const float* cos_t, const float* sin_t, int rot_dims, const int* positions,
-                                const float* pre, cudaStream_t stream) {
+                                const float* pre, int pairing, cudaStream_t stream) {
   if (T <= 0) return 0;
   size_t smem = (size_t)LA_TT * dn * sizeof(float);
   if (smem > 48 * 1024 || H > 65535) return QD_ERR_UNSUPPORTED;
@@ -647,20 +638,20 @@ extern "C" int qd_latent_absorb(const float* q, long long ldq, const void* wuk, 
       dim3 vgrid((T + LA_TT - 1) / LA_TT, H);
       if (w_dtype == QD_F32)
         qd_launch(latent_absorb_vec_kernel<float>, vgrid, dim3(256), vsm, stream, q, ldq, (const float*)wuk, qcat, T, H, dn, dr,
-                  r, cos_t, sin_t, rot_dims, positions);
+                  r, cos_t, sin_t, rot_dims, positions, pairing);
       else
         qd_launch(latent_absorb_vec_kernel<bf16>, vgrid, dim3(256), vsm, stream, q, ldq, (const bf16*)wuk, qcat, T, H, dn, dr,
-                  r, cos_t, sin_t, rot_dims, positions);
+                  r, cos_t, sin_t, rot_dims, positions, pairing);
       return qd_last_error();
     }
   }
   dim3 grid((T + LA_TT - 1) / LA_TT, H, (r + 255) / 256);
   if (w_dtype == QD_F32)
     qd_launch(latent_absorb_kernel<float>, grid, dim3(256), smem, stream, q, ldq, (const float*)wuk, qcat, T, H, dn, dr, r,
-              cos_t, sin_t, rot_dims, positions, pre);
+              cos_t, sin_t, rot_dims, positions, pre, pairing);
   else if (w_dtype == QD_BF16)
     qd_launch(latent_absorb_kernel<bf16>, grid, dim3(256), smem, stream, q, ldq, (const bf16*)wuk, qcat, T, H, dn, dr, r,
-              cos_t, sin_t, rot_dims, positions, pre);
+              cos_t, sin_t, rot_dims, positions, pre, pairing);
   else
     return QD_ERR_UNSUPPORTED;
   return qd_last_error();

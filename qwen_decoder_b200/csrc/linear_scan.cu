@@ -13,8 +13,16 @@
 //              S <- g S;   x = v, or with the delta rule x = beta (v - S^T k);   S <- S + k x^T;   o = S^T q
 //            S lives in the request's state row as [H, dv, d] (a value column's d elements side by side), float32, read
 //            and written once per step
-//   finish   out[t, h] = o / sqrt(mean(o^2) + eps) (* norm [dv]) * silu(gate) * out_scale, rounded once
+//   finish   out[t, h] = o / sqrt(mean(o^2) + eps) (* norm) * silu(gate) (or sigmoid) * out_scale, rounded once
 //   step     scan and finish of single tokens, one per request, in one launch: a CTA owns a whole head
+//
+// With exponential gates (``ExpGates``) a head has a log input gate i = cap tanh((u_i + ib) / cap), a log forget gate
+// f = logsigmoid(cap tanh((u_f + fb) / cap)) and a running maximum m (0 for a fresh request), m' = max(f + m, i):
+//   S <- e^(f + m - m') S + e^(i - m') k v^T,   n <- e^(f + m - m') n + e^(i - m') k,
+//   o = S^T q / (max(|n . q|, e^-m') + 1e-6)
+// n is one more column of S whose value is always 1 (the state then is [H, dv + 1, d], and m is kept beside it);
+// ``gates`` makes the decays, e^(i - m') and e^-m' of portions, ``prep`` multiplies k by e^(i - m'), ``finish`` divides.
+// A step of single tokens does all of it in its one launch.
 //
 // Everything is float32 until ``finish``'s store.  The order of every sum depends on the sizes and on a token's place in its
 // portion only: however a prompt is cut, the results agree up to the rounding of float32 sums.
@@ -27,6 +35,8 @@ __device__ __forceinline__ void ls_st(void* p, int code, size_t i, float v) {
   else reinterpret_cast<bf16*>(p)[i] = __float2bfloat16_rn(v);
 }
 __device__ __forceinline__ float ls_silu(float z) { return z / (1.0f + expf(-z)); }
+// What the output gate multiplies by: silu (0) or sigmoid (1) of the logit.
+__device__ __forceinline__ float ls_gate(float z, int kind) { return (kind ? 1.0f : z) / (1.0f + expf(-z)); }
 __device__ __forceinline__ float ls_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 
 // ------------------------------------------------------------------------------------------------------------ prep
@@ -43,6 +53,7 @@ struct LinearPrep {
   int rotary_dim, pairing; const float *cos_t, *sin_t; const int* positions;
   float q_scale, k_scale;
   int b_off, a_off; const float *A_log, *dt_bias;             // columns of u, -1: not there
+  const float* k_mul;                                          // [T, G]: one more factor of k, or null
   float *q, *k, *v, *beta, *g;                                 // [T, G, DP] twice, [T, H * dv], [T, H] twice
   int v_slots, tokens;
 };
@@ -117,6 +128,7 @@ linear_prep_kernel(LinearPrep a) {
       for (int i = lane; i < d; i += 32) ss = fmaf(lp_sm[tt * d + i], lp_sm[tt * d + i], ss);
       c *= 1.0f / sqrtf(warp_sum(ss) + a.unit_eps);
     }
+    if (!is_q && a.k_mul) c *= a.k_mul[(size_t)(t0 + tt) * a.G + head];
     if (lane == 0) f[tt] = c;
   }
   __syncthreads();
@@ -157,14 +169,14 @@ linear_prep_state_kernel(const float* __restrict__ u, long long ld, int C, int t
 // u float32 [T, ld], a row = [q (G*d) | k (G*d) | v (H*dv) | ...]; conv_w float32 [2*G*d + H*dv, taps] (taps 0: no
 // convolution, no silu, and v is not written); state rows ``state_stride`` apart with the (taps - 1) x C kept inputs at
 // ``conv_off``, moved on by the portions when ``update_state``; b_off / a_off: columns of u of the step size's and the
-// decay's logits (-1: none).
+// decay's logits (-1: none); k_mul float32 [T, G] (null: none): multiplies k's heads.
 extern "C" int qd_linear_prep(const float* u, long long ld, int T, int n_requests, int H, int G, int d, int dv, int DP,
                               int taps, const float* conv_w, float* state, long long state_stride, long long conv_off,
                               const int* token_req, const int* cu_tokens, const int* slots, int update_state, int unit,
                               float unit_eps, int rotary_dim, int pairing, const float* cos_t, const float* sin_t,
                               const int* positions, float q_scale, float k_scale, int b_off, int a_off,
-                              const float* A_log, const float* dt_bias, float* q, float* k, float* v, float* beta,
-                              float* g, cudaStream_t stream) {
+                              const float* A_log, const float* dt_bias, const float* k_mul, float* q, float* k, float* v,
+                              float* beta, float* g, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || d <= 0 || dv <= 0 || DP < d || DP > 256 || taps < 0 || (taps > 0 && (!conv_w || !v)) ||
       (taps > 1 && !state) || rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1) ||
@@ -187,13 +199,103 @@ extern "C" int qd_linear_prep(const float* u, long long ld, int T, int n_request
   const int advance = update_state && taps > 1 && T == n_requests;       // single tokens, one per request
   const LinearPrep a = {u, ld, T, H, G, d, dv, DP, taps, conv_w, state, state_stride, conv_off, advance, token_req, cu_tokens,
                         slots, unit, unit_eps, rotary_dim, pairing, cos_t, sin_t, positions, q_scale, k_scale, b_off, a_off,
-                        A_log, dt_bias, q, k, v, beta, g, v_slots, tokens};
+                        A_log, dt_bias, k_mul, q, k, v, beta, g, v_slots, tokens};
   qd_launch(linear_prep_kernel, dim3(slots_x, (T + tokens - 1) / tokens), dim3(LP_THREADS), smem, stream, a);
   if (update_state && taps > 1 && !advance) {
     const int C = 2 * G * d + H * dv;
     qd_launch(linear_prep_state_kernel, dim3((C + 255) / 256, n_requests), dim3(256), 0, stream, u, ld, C, taps, state,
               state_stride, conv_off, cu_tokens, slots);
   }
+  return qd_last_error();
+}
+
+// ----------------------------------------------------------------------------------------------- exponential gates
+#define LS_NRM_EPS 1e-6f      // beside the larger of |n . q| and e^-m in the denominator
+struct ExpGates {
+  const float* u; long long ld; int i_off, f_off;             // the logits: row t at t * ld, head h at i_off + h, f_off + h
+  const float *ib, *fb; float cap;                            // [H] each
+  long long m_off;                                            // head h's maximum is at m_off + h of a state row
+  int on;
+};
+__device__ __forceinline__ void exp_gate_logs(const ExpGates& a, int t, int h, float& i, float& f) {
+  const float* row = a.u + (size_t)t * a.ld;
+  i = a.cap * tanhf((row[a.i_off + h] + a.ib[h]) / a.cap);
+  const float z = a.cap * tanhf((row[a.f_off + h] + a.fb[h]) / a.cap);
+  f = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+}
+
+// grid (H, requests), one warp: the maxima of a portion by a scan over (sum of f, maximum): what a run of tokens does to m is
+// m -> max(F + m, M), and runs compose.  A lane takes LG_RUN neighbouring tokens.  Every factor is made from the maxima as
+// they are handed on, so what rounds in the scan cancels between a token and the next.
+#define LG_RUN 8
+__global__ void __launch_bounds__(32)
+linear_exp_gates_kernel(ExpGates a, int H, float* __restrict__ state, long long state_stride,
+                        const int* __restrict__ cu_tokens, const int* __restrict__ slots, int write_state,
+                        float* __restrict__ g, float* __restrict__ in, float* __restrict__ low) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.x, req = blockIdx.y, lane = threadIdx.x;
+  const int t0 = cu_tokens[req], t1 = cu_tokens[req + 1];
+  if (t0 >= t1) return;
+  float* kept = state + (size_t)slots[req] * state_stride + a.m_off + h;
+  float m0 = *kept;
+  for (int tb = t0; tb < t1; tb += 32 * LG_RUN) {
+    float iv[LG_RUN], fv[LG_RUN], F = 0.f, M = -INFINITY;
+#pragma unroll
+    for (int j = 0; j < LG_RUN; j++) {
+      const int t = tb + lane * LG_RUN + j;
+      iv[j] = -INFINITY;                              // past the end: m stays as it is
+      fv[j] = 0.f;
+      if (t < t1) exp_gate_logs(a, t, h, iv[j], fv[j]);
+      F += fv[j];
+      M = fmaxf(M + fv[j], iv[j]);
+    }
+    float Fs = F, Ms = M;                             // of all lanes up to this one
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float Fp = __shfl_up_sync(0xffffffffu, Fs, o), Mp = __shfl_up_sync(0xffffffffu, Ms, o);
+      if (lane >= o) {
+        Ms = fmaxf(Mp + Fs, Ms);
+        Fs += Fp;
+      }
+    }
+    float Fb = __shfl_up_sync(0xffffffffu, Fs, 1), Mb = __shfl_up_sync(0xffffffffu, Ms, 1);
+    float m = lane ? fmaxf(Fb + m0, Mb) : m0;         // before this lane's run
+    float mv[LG_RUN];
+#pragma unroll
+    for (int j = 0; j < LG_RUN; j++) {
+      m = fmaxf(fv[j] + m, iv[j]);
+      mv[j] = m;
+    }
+    float before = __shfl_up_sync(0xffffffffu, m, 1); // as the lane before hands it on
+    if (!lane) before = m0;
+#pragma unroll
+    for (int j = 0; j < LG_RUN; j++) {
+      const int t = tb + lane * LG_RUN + j;
+      if (t < t1) {
+        const size_t at = (size_t)t * H + h;
+        g[at] = expf(fv[j] + (before - mv[j]));
+        in[at] = expf(iv[j] - mv[j]);
+        low[at] = expf(-mv[j]);
+      }
+      before = mv[j];
+    }
+    m0 = __shfl_sync(0xffffffffu, m, 31);
+  }
+  if (write_state && lane == 0) *kept = m0;
+}
+
+// From the logits' columns of u: g = e^(f + m - m'), in = e^(i - m') and low = e^-m', float32 [T, H]; the maxima of the
+// requests' state rows are moved on when ``write_state``.
+extern "C" int qd_linear_exp_gates(const float* u, long long ld, int i_off, int f_off, const float* ib, const float* fb,
+                                   float cap, int T, int n_requests, int H, float* state, long long state_stride,
+                                   long long m_off, const int* cu_tokens, const int* slots, int write_state, float* g,
+                                   float* in, float* low, cudaStream_t stream) {
+  if (T <= 0 || n_requests <= 0) return 0;
+  if (H <= 0 || n_requests > 65535 || !ib || !fb || !(cap > 0.f) || !state || !g || !in || !low) return QD_ERR_UNSUPPORTED;
+  const ExpGates a = {u, ld, i_off, f_off, ib, fb, cap, m_off, 1};
+  qd_launch(linear_exp_gates_kernel, dim3(H, n_requests), dim3(32), 0, stream, a, H, state, state_stride, cu_tokens, slots,
+            write_state, g, in, low);
   return qd_last_error();
 }
 
@@ -210,6 +312,9 @@ struct LinearScan {
   float* state; long long state_stride, s_off; int vec;         // vec: rows of d elements start on 16-byte boundaries
   const int *cu_tokens, *slots;
   int write_state;
+  int nrm; float* nq;                     // nrm: one more column whose value is 1; its outputs [T, H]
+  // single tokens: where q's and k's rows are, if they are not padded (``raw``), and what they are still multiplied by
+  int raw; long long q_ld; float q_scale, k_scale;
 };
 
 // Two float32 numbers that one instruction works on (each rounded as by itself).
@@ -361,7 +466,8 @@ __device__ __forceinline__ void ls_fetch(const LinearScan& a, float* st, int tb,
   for (int e = tid; e < LS_GROUP * COLS; e += THREADS) {
     const int tt = e / COLS, c = e - tt * COLS;
     const bool there = tb + tt < t1 && j0 + c < a.dv;
-    ls_cp4(st + L::V + e, there ? a.v + (size_t)(tb + tt) * a.ldv + (size_t)h * a.dv + j0 + c : a.v, there);
+    if (!DELTA && a.nrm && j0 + c == a.dv) st[L::V + e] = tb + tt < t1 ? 1.0f : 0.0f;
+    else ls_cp4(st + L::V + e, there ? a.v + (size_t)(tb + tt) * a.ldv + (size_t)h * a.dv + j0 + c : a.v, there);
   }
   if (DELTA) {
     if (tid < LS_GROUP * (LS_COEF / 4)) {
@@ -390,14 +496,15 @@ linear_scan_kernel(LinearScan a, float* __restrict__ out) {
   extern __shared__ __align__(16) float ls_sm[];      // two stages
   const int tid = threadIdx.x, x = tid & 7, jl = (tid >> 3) * CPT;
   const int h = blockIdx.y, req = blockIdx.z, j0 = blockIdx.x * COLS, j = j0 + jl;
-  const int gk = h / (a.H / a.G), d = a.d, dv = a.dv;
+  const int gk = h / (a.H / a.G), d = a.d, dv = a.dv, nc = dv + a.nrm;
   const int t0 = a.cu_tokens[req], t1 = a.cu_tokens[req + 1];
   if (t0 >= t1) return;
-  float* S = a.state + (size_t)a.slots[req] * a.state_stride + a.s_off + (size_t)h * dv * d;
+  float* S = a.state + (size_t)a.slots[req] * a.state_stride + a.s_off + (size_t)h * nc * d;
   ls_fetch<DP, false, COLS, THREADS>(a, ls_sm, t0, t1, h, gk, j0);
+  const bool busy = j0 + (tid >> 5) * 4 * CPT < nc;   // whether this warp has a column at all
   f2 s[CPT][E / 2];
 #pragma unroll
-  for (int c = 0; c < CPT; c++) ls_load_state<E, 8>(s[c], S + (size_t)(j + c < dv ? j + c : 0) * d, x, d, j + c < dv, a.vec);
+  for (int c = 0; c < CPT; c++) ls_load_state<E, 8>(s[c], S + (size_t)(j + c < nc ? j + c : 0) * d, x, d, j + c < nc, a.vec);
   int stage = 0;
   for (int tb = t0; tb < t1; tb += LS_GROUP, stage ^= 1) {
     if (tb + LS_GROUP < t1) {
@@ -408,7 +515,7 @@ linear_scan_kernel(LinearScan a, float* __restrict__ out) {
     }
     __syncthreads();
     const float* st = ls_sm + stage * L::FLOATS;
-    const int nt = min(LS_GROUP, t1 - tb);
+    const int nt = busy ? min(LS_GROUP, t1 - tb) : 0;
     for (int b = 0; b < nt; b += RUN) {
       float acc[8];                                   // token b + p, column jl + c: this thread's share at CPT p + c
 #pragma unroll
@@ -427,13 +534,14 @@ linear_scan_kernel(LinearScan a, float* __restrict__ out) {
       const float o = ls_reduce<8>(acc, x);
       const int tt = b + x / CPT, c = j + x % CPT;
       if (tt < nt && c < dv) out[(size_t)(tb + tt) * a.H * dv + (size_t)h * dv + c] = o;
+      else if (tt < nt && c < nc) a.nq[(size_t)(tb + tt) * a.H + h] = o;
     }
     __syncthreads();                                  // this stage is overwritten by the next turn's fetch
   }
   if (!a.write_state) return;
 #pragma unroll
   for (int c = 0; c < CPT; c++)
-    if (j + c < dv) ls_store_state<E, 8>(s[c], S + (size_t)(j + c) * d, x, d, a.vec);
+    if (j + c < nc) ls_store_state<E, 8>(s[c], S + (size_t)(j + c) * d, x, d, a.vec);
 }
 
 // The delta rule in runs of four tokens.  With S0 the state before a run, G_p = g_0 .. g_p and d(s, p) = g_(s+1) .. g_p,
@@ -600,9 +708,11 @@ linear_delta_kernel(LinearScan a, float* __restrict__ out) {
 
 // ---------------------------------------------------------------------------------------------------------- finish
 struct LinearFinish {
-  const float* gate; long long gate_ld;   // float32 logits, head h's at + h * dv; silu is taken here
-  const float* norm;                      // [dv] or null
+  const float* gate; long long gate_ld;   // float32 logits, head h's at + h * dv; silu or sigmoid (``gate_kind`` 1) is taken here
+  const float* norm; int norm_ld;         // [dv] (norm_ld 0) or [H, dv] (norm_ld dv), or null
   float eps, out_scale;
+  int gate_kind;
+  const float *nq, *low;                  // [T, H]: o is first divided by max(|nq|, low) + LS_NRM_EPS; or null
   void* out; int out_dtype; long long out_stride;
 };
 
@@ -634,17 +744,25 @@ linear_finish_kernel(const float* __restrict__ o, int T, int H, int dv, LinearFi
 #pragma unroll
   for (int s = LANES / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
   if (!there) return;
-  const float c = f.out_scale / sqrtf(ss / (float)dv + f.eps);
+  const float* norm = f.norm ? f.norm + (size_t)h * f.norm_ld : nullptr;
+  float c = f.out_scale;
+  if (f.nq) {
+    const float r = 1.0f / (fmaxf(fabsf(f.nq[item]), f.low[item]) + LS_NRM_EPS);
+    ss *= r * r;
+    c *= r;
+  }
+  c /= sqrtf(ss / (float)dv + f.eps);
   if (vec) {
     for (int i = lane * 4; i < dv; i += LANES * 4) {
       const float4 y = i == lane * 4 ? first : *reinterpret_cast<const float4*>(row + i);
       const float4 z = *reinterpret_cast<const float4*>(gate + i);
       float4 n = make_float4(c, c, c, c);
-      if (f.norm) {
-        const float4 w = *reinterpret_cast<const float4*>(f.norm + i);
+      if (norm) {
+        const float4 w = *reinterpret_cast<const float4*>(norm + i);
         n = make_float4(c * w.x, c * w.y, c * w.z, c * w.w);
       }
-      const float4 r = make_float4(y.x * n.x * ls_silu(z.x), y.y * n.y * ls_silu(z.y), y.z * n.z * ls_silu(z.z), y.w * n.w * ls_silu(z.w));
+      const float4 r = make_float4(y.x * n.x * ls_gate(z.x, f.gate_kind), y.y * n.y * ls_gate(z.y, f.gate_kind),
+                                   y.z * n.z * ls_gate(z.z, f.gate_kind), y.w * n.w * ls_gate(z.w, f.gate_kind));
       if (f.out_dtype == QD_F32) {
         *reinterpret_cast<float4*>(reinterpret_cast<float*>(f.out) + dst + i) = r;
       } else {
@@ -658,85 +776,137 @@ linear_finish_kernel(const float* __restrict__ o, int T, int H, int dv, LinearFi
     return;
   }
   for (int i = lane; i < dv; i += LANES)
-    ls_st(f.out, f.out_dtype, dst + i, row[i] * c * (f.norm ? f.norm[i] : 1.0f) * ls_silu(gate[i]));
+    ls_st(f.out, f.out_dtype, dst + i, row[i] * c * (norm ? norm[i] : 1.0f) * ls_gate(gate[i], f.gate_kind));
 }
 
 // ------------------------------------------------------------------------------------------------------------ step
-// grid (H, requests), 4 * (columns at a time) threads, at most 512: four neighbouring lanes to a value column.  Request r's
-// token is token r.
-#define LS_STEP_THREADS 512
+// grid (H, requests), 4 * (columns at a time) threads, at most LS_STEP_THREADS: four neighbouring lanes to a value column.
+// Request r's token is token r.
+#define LS_STEP_THREADS(DP) ((DP) > 128 ? 256 : 512)
+
+// A lane's elements of a row of q or k: padded rows, or (``raw``) rows of d numbers where they stand.
+template <int E>
+__device__ __forceinline__ void ls_step_row(f2 (&r)[E / 2], const float* row, int x, int d, int raw, int vec, float scale) {
+  if (!raw) {
+    ls_row<E, 4>(r, row, x);
+    return;
+  }
+  ls_load_state<E, 4>(r, row, x, d, true, vec);
+  const f2 c = f2_make(scale, scale);
+#pragma unroll
+  for (int m = 0; m < E / 2; m++) r[m] = f2_mul<false>(r[m], c);
+}
 
 template <int DP, bool DELTA>
-__global__ void __launch_bounds__(LS_STEP_THREADS)
-linear_step_kernel(LinearScan a, LinearFinish f) {
+__global__ void __launch_bounds__(LS_STEP_THREADS(DP))
+linear_step_kernel(LinearScan a, LinearFinish f, ExpGates eg) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int E = DP / 4;
-  extern __shared__ float st_sm[];                    // [dv] outputs, then 40 of scratch
+  extern __shared__ float st_sm[];                    // [dv + nrm] outputs, then 40 of scratch
   const int tid = threadIdx.x, x = tid & 3, jl = tid >> 2, cols = blockDim.x >> 2;
-  const int h = blockIdx.x, t = blockIdx.y, d = a.d, dv = a.dv, gk = h / (a.H / a.G);
-  float* S = a.state + (size_t)a.slots[t] * a.state_stride + a.s_off + (size_t)h * dv * d;
-  const float* kr = a.k + ((size_t)t * a.G + gk) * DP;
-  const float* qr = a.q + ((size_t)t * a.G + gk) * DP;
-  const float g = a.g[(a.g_ld ? (size_t)t * a.g_ld : 0) + h];
+  const int h = blockIdx.x, t = blockIdx.y, d = a.d, dv = a.dv, nc = dv + a.nrm, gk = h / (a.H / a.G);
+  float* kept = a.state + (size_t)a.slots[t] * a.state_stride;
+  float* S = kept + a.s_off + (size_t)h * nc * d;
+  const long long q_ld = a.raw ? a.q_ld : (long long)a.G * DP;
+  const float* kr = a.k + (size_t)t * q_ld + (size_t)gk * (a.raw ? d : DP);
+  const float* qr = a.q + (size_t)t * q_ld + (size_t)gk * (a.raw ? d : DP);
+  const int qvec = a.vec && q_ld % 4 == 0 && !(((uintptr_t)a.q | (uintptr_t)a.k) & 15);
+  float g, in = 1.f, m = 0.f;
+  if (!DELTA && eg.on) {
+    float i, lf;
+    exp_gate_logs(eg, t, h, i, lf);
+    const float m0 = kept[eg.m_off + h];
+    m = fmaxf(lf + m0, i);
+    g = expf(lf + (m0 - m));
+    in = expf(i - m);
+  } else {
+    g = a.g[(a.g_ld ? (size_t)t * a.g_ld : 0) + h];
+  }
   const float beta = DELTA ? a.beta[(size_t)t * a.H + h] : 0.f;
   float ss = 0.f;
-  for (int j0 = 0; j0 < dv; j0 += cols) {             // every thread takes every turn: the shuffles need them all
+  for (int j0 = 0; j0 < nc; j0 += cols) {             // every thread takes every turn: the shuffles need them all
     const int j = j0 + jl;
-    const bool live = j < dv;
+    const bool live = j < nc;
     float* col = S + (size_t)(live ? j : 0) * d;
     f2 s[E / 2];
     ls_load_state<E, 4>(s, col, x, d, live, a.vec);
-    float w = live ? a.v[(size_t)t * a.ldv + (size_t)h * dv + j] : 0.f;
+    float w = j < dv ? a.v[(size_t)t * a.ldv + (size_t)h * dv + j] : live ? 1.f : 0.f;
     f2 r[E / 2];
-    ls_row<E, 4>(r, kr, x);
+    ls_step_row<E>(r, kr, x, d, a.raw, qvec, a.k_scale);
     if (DELTA) {
       float dot = ls_dot<E, false>(s, r);
       dot += __shfl_xor_sync(0xffffffffu, dot, 2);
       dot += __shfl_xor_sync(0xffffffffu, dot, 1);
       w = beta * fmaf(-g, dot, w);
+    } else {
+      w *= in;
     }
     ls_move<E, false>(s, r, w, g);
-    ls_row<E, 4>(r, qr, x);
+    ls_step_row<E>(r, qr, x, d, a.raw, qvec, a.q_scale);
     float o = ls_dot<E, false>(s, r);
     o += __shfl_xor_sync(0xffffffffu, o, 2);
     o += __shfl_xor_sync(0xffffffffu, o, 1);
     if (live && x == 0) {
       st_sm[j] = o;
-      ss = fmaf(o, o, ss);
+      if (j < dv) ss = fmaf(o, o, ss);
     }
     if (a.write_state && live) ls_store_state<E, 4>(s, col, x, d, a.vec);
   }
-  const float c = f.out_scale / sqrtf(block_sum(ss, st_sm + dv) / (float)dv + f.eps);     // meets the writes of st_sm, too
+  ss = block_sum(ss, st_sm + nc);                     // meets the writes of st_sm and every thread's read of the maximum, too
+  float c = f.out_scale;
+  if (a.nrm) {
+    const float r = 1.0f / (fmaxf(fabsf(st_sm[dv]), expf(-m)) + LS_NRM_EPS);
+    ss *= r * r;
+    c *= r;
+  }
+  c /= sqrtf(ss / (float)dv + f.eps);
+  if (!DELTA && eg.on && a.write_state && tid == 0) kept[eg.m_off + h] = m;
   const float* gate = f.gate + (size_t)t * f.gate_ld + (size_t)h * dv;
+  const float* norm = f.norm ? f.norm + (size_t)h * f.norm_ld : nullptr;
   for (int i = tid; i < dv; i += blockDim.x)
     ls_st(f.out, f.out_dtype, (size_t)t * f.out_stride + (size_t)h * dv + i,
-          st_sm[i] * c * (f.norm ? f.norm[i] : 1.0f) * ls_silu(gate[i]));
+          st_sm[i] * c * (norm ? norm[i] : 1.0f) * ls_gate(gate[i], f.gate_kind));
 }
 
 // ------------------------------------------------------------------------------------------------------- launchers
 // q, k float32 [T, G, DP], DP the padded head size: the smallest of 32, 64, 96, 128, 256 that holds d; v rows
 // ``ldv`` apart; g float32 [T, H] (g_ld = H) or [H] (g_ld = 0); beta float32 [T, H]: the delta rule, or null;
 // state float32 rows ``state_stride`` apart, the heads' matrices [H, dv, d] at ``s_off``; o_buf float32 [T, H * dv]
-// (unused when every request brings one token); coef float32 [T, H, LS_COEF] of scratch for the delta rule (unused then, too); gate float32 rows ``gate_ld`` apart; norm float32 [dv] or null.
+// (unused when every request brings one token); coef float32 [T, H, LS_COEF] of scratch for the delta rule (unused then, too);
+// gate float32 rows ``gate_ld`` apart; norm float32 [dv] (norm_ld 0) or [H, dv] (norm_ld dv), or null; gate_kind 0 silu, 1 sigmoid.
+// ``nrm``: exponential gates.  S is [H, dv + 1, d] at ``s_off``, the maxima at ``m_off``; portions: nq scratch [T, H], g, low and k
+// as ``qd_linear_exp_gates`` and ``qd_linear_prep`` made them; single tokens: g unused, the logits are columns i_off, f_off of u.
+// ``raw`` (single tokens): q and k are rows of G * d numbers ``q_ld`` apart that q_scale and k_scale still multiply.
 extern "C" int qd_linear_scan(const float* q, const float* k, const float* v, long long ldv, const float* g, int g_ld,
                               const float* beta, int T, int n_requests, int H, int G, int d, int dv, int DP,
                               float* state, long long state_stride, long long s_off, const int* cu_tokens,
                               const int* slots, int write_state, float* o_buf, const float* gate, long long gate_ld,
                               const float* norm, float eps, float out_scale, void* out, int out_dtype,
-                              long long out_stride, const int* token_req, float* coef, cudaStream_t stream) {
+                              long long out_stride, const int* token_req, float* coef, int norm_ld, int gate_kind, int nrm,
+                              float* nq, const float* low, const float* u, long long u_ld, int i_off, int f_off,
+                              const float* ib, const float* fb, float cap, long long m_off, int raw, long long q_ld,
+                              float q_scale, float k_scale, cudaStream_t stream) {
   if (T <= 0 || n_requests <= 0) return 0;
   if (H <= 0 || H > 65535 || n_requests > 65535 || G <= 0 || H % G || d <= 0 || dv <= 0 || dv > 8192 || d > DP ||
       !state || !gate || (g_ld && g_ld != H) || (beta && T != n_requests && (!coef || ((uintptr_t)coef & 15))) || (out_dtype != QD_F32 && out_dtype != QD_BF16))
     return QD_ERR_UNSUPPORTED;
   const bool single = T == n_requests;                // every request has at least one token
   if (!single && !o_buf) return QD_ERR_UNSUPPORTED;
-  if (((uintptr_t)q | (uintptr_t)k) & 15) return QD_ERR_UNSUPPORTED;
+  if (nrm && (beta || G != H || (single ? !u || !ib || !fb || !(cap > 0.f) : !nq || !low))) return QD_ERR_UNSUPPORTED;
+  if (raw ? !single : (((uintptr_t)q | (uintptr_t)k) & 15) != 0) return QD_ERR_UNSUPPORTED;
+  if (!g && !(nrm && single)) return QD_ERR_UNSUPPORTED;
+  nrm = nrm ? 1 : 0;
+  const int nc = dv + nrm;
   const int vec = d % 4 == 0 && state_stride % 4 == 0 && s_off % 4 == 0 && !((uintptr_t)state & 15);
-  const LinearScan a = {q, k, v, ldv, g, g_ld, beta, coef, H, G, d, dv, state, state_stride, s_off, vec, cu_tokens, slots, write_state};
-  const LinearFinish f = {gate, gate_ld, norm, eps, out_scale, out, out_dtype, out_stride};
-  const int cols = (dv + 7) / 8 * 8 < LS_STEP_THREADS / 4 ? (dv + 7) / 8 * 8 : LS_STEP_THREADS / 4;
-  const size_t step_smem = ((size_t)dv + 40) * sizeof(float);
+  const LinearScan a = {q, k, v, ldv, g, g_ld, beta, coef, H, G, d, dv, state, state_stride, s_off, vec, cu_tokens, slots,
+                        write_state, nrm, nq, raw, q_ld, q_scale, k_scale};
+  const LinearFinish f = {gate, gate_ld, norm, norm_ld, eps, out_scale, gate_kind, nrm ? nq : nullptr, low, out, out_dtype,
+                          out_stride};
+  const ExpGates eg = {u, u_ld, i_off, f_off, ib, fb, cap, m_off, nrm};
+  // as many columns at a time as make the turns even
+  const int most = LS_STEP_THREADS(DP) / 4, turns = (nc + most - 1) / most, cols = ((nc + turns - 1) / turns + 7) / 8 * 8;
+  const size_t step_smem = ((size_t)nc + 40) * sizeof(float);
   // few heads: half as many columns to a CTA, so that more multiprocessors work
   static int sms = 0;
   if (!sms) {
@@ -744,7 +914,7 @@ extern "C" int qd_linear_scan(const float* q, const float* k, const float* v, lo
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   }
-  const bool narrow = (long long)((dv + 31) / 32) * H * n_requests * 2 <= sms + sms / 8;
+  const bool narrow = (long long)((nc + 31) / 32) * H * n_requests * 2 <= sms + sms / 8;
 #define LS_LAUNCH(KERNEL, COLS, THREADS, FLOATS)                                                                     \
   do {                                                                                                                \
     const size_t smem = (size_t)(FLOATS) * sizeof(float);                                                             \
@@ -756,12 +926,12 @@ extern "C" int qd_linear_scan(const float* q, const float* k, const float* v, lo
     /* The scan's CTAs are few and long: launched while the kernel before them still runs they would crowd onto the   \
        multiprocessors that become free first. */                                                                     \
     qd_plain_next_launch = true;                                                                                      \
-    qd_launch(KERNEL, dim3((dv + COLS - 1) / COLS, H, n_requests), dim3(THREADS), smem, stream, a, o_buf);             \
+    qd_launch(KERNEL, dim3((nc + COLS - 1) / COLS, H, n_requests), dim3(THREADS), smem, stream, a, o_buf);             \
   } while (0)
 #define LS_DELTA(DP)                                                                                                  \
   do {                                                                                                                \
     if (single) {                                                                                                     \
-      qd_launch(linear_step_kernel<DP, true>, dim3(H, n_requests), dim3(4 * cols), step_smem, stream, a, f);          \
+      qd_launch(linear_step_kernel<DP, true>, dim3(H, n_requests), dim3(4 * cols), step_smem, stream, a, f, eg);          \
       break;                                                                                                          \
     }                                                                                                                 \
     qd_launch(linear_coef_kernel<DP>, dim3((unsigned)(((long long)T * G + 7) / 8)), dim3(256), 0, stream, q, k, g, g_ld, \
@@ -772,7 +942,7 @@ extern "C" int qd_linear_scan(const float* q, const float* k, const float* v, lo
   } while (0)
 #define LS_PLAIN(DP)                                                                                                  \
   do {                                                                                                                \
-    if (single) qd_launch(linear_step_kernel<DP, false>, dim3(H, n_requests), dim3(4 * cols), step_smem, stream, a, f); \
+    if (single) qd_launch(linear_step_kernel<DP, false>, dim3(H, n_requests), dim3(4 * cols), step_smem, stream, a, f, eg); \
     else if (narrow) LS_LAUNCH((linear_scan_kernel<DP, 16, 1>), 16, 128, (2 * LsStage<DP, false, 16>::FLOATS));        \
     else LS_LAUNCH((linear_scan_kernel<DP, 32, 2>), 32, 128, (2 * LsStage<DP, false, 32>::FLOATS));                    \
   } while (0)

@@ -15,7 +15,8 @@
 // min(g, L) * sigmoid(a * min(g, L)) * (clamp(u, -L, L) + 1) (``act`` 1) instead of silu(g) * u.  ``route_mode`` 2 chooses
 // the ``top`` largest logits and weighs each by its own sigmoid, not renormalised.  A pair's weight may multiply the
 // expert's INPUT instead of its output (``in_scale`` of the gated product: W (w h) = w (W h), so both sums of the pair
-// are multiplied by w before the gate; combine then adds the pairs' outputs as they are).
+// are multiplied by w before the gate; combine then adds the pairs' outputs as they are).  ``route_mode`` 3 chooses as 2
+// does and divides the chosen sigmoids by their sum + 1e-20; every mode's weights are multiplied by ``scale``.
 //
 // Nothing comes back to the host between these: counts, places and tiles stay on the device, so a step with
 // routed experts is captured in a CUDA graph like any other.  The products run on float32 FMA with the
@@ -24,10 +25,10 @@
 
 #define MOE_MAX_TOP 32
 
-// The gate of a gated expert: act 0 silu(g) * u; act 1 the clamped form with slope ``alpha`` and limit ``limit``.
+// The gate of a gated expert: act 0 silu(g) * u, 2 gelu(g) * u; act 1 the clamped form with slope ``alpha`` and limit ``limit``.
 struct MoeAct { int kind; float limit, alpha; };
 __device__ __forceinline__ float moe_gated(float g, float u, MoeAct a) {
-  if (a.kind == 0) return g / (1.0f + expf(-g)) * u;
+  if (a.kind != 1) return qd_gated(g, u, a.kind);
   g = fminf(g, a.limit);
   u = fminf(fmaxf(u, -a.limit), a.limit);
   return g / (1.0f + expf(-a.alpha * g)) * (u + 1.0f);
@@ -107,7 +108,7 @@ moe_logits_kernel(const T* __restrict__ h, const T* __restrict__ wr, const float
 // weighed by sigmoid(logit).
 __global__ void __launch_bounds__(128)
 moe_topk_kernel(float* __restrict__ logits, int n_tokens, int E, int top, int mode, const float* __restrict__ corr,
-                int* __restrict__ idx, float* __restrict__ wt) {
+                int* __restrict__ idx, float* __restrict__ wt, float scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x * blockDim.x + threadIdx.x;
@@ -130,7 +131,7 @@ moe_topk_kernel(float* __restrict__ logits, int n_tokens, int E, int top, int mo
         if (best < 0 || c > bv) { best = e; bv = c; }
       }
       idx[(size_t)t * top + k] = best;
-      wt[(size_t)t * top + k] = my[best];
+      wt[(size_t)t * top + k] = my[best] * scale;
       my[best] = -1.0f;
     }
     return;
@@ -146,14 +147,16 @@ moe_topk_kernel(float* __restrict__ logits, int n_tokens, int E, int top, int mo
     v[k] = bv;
     my[best] = -INFINITY;
   }
-  if (mode == 2) {                                // each chosen output's own sigmoid
-    for (int k = 0; k < top; k++) wt[(size_t)t * top + k] = 1.0f / (1.0f + expf(-v[k]));
+  float sum = 0.f;
+  if (mode >= 2) {                                // each chosen output's own sigmoid, in mode 3 divided by their sum
+    for (int k = 0; k < top; k++) { v[k] = 1.0f / (1.0f + expf(-v[k])); sum += v[k]; }
+    const float f = mode == 3 ? scale / (sum + 1e-20f) : scale;
+    for (int k = 0; k < top; k++) wt[(size_t)t * top + k] = v[k] * f;
     return;
   }
-  float sum = 0.f;
   const float vmax = v[0];                        // the first chosen is the largest
   for (int k = 0; k < top; k++) { v[k] = expf(v[k] - vmax); sum += v[k]; }
-  for (int k = 0; k < top; k++) wt[(size_t)t * top + k] = v[k] / sum;
+  for (int k = 0; k < top; k++) wt[(size_t)t * top + k] = v[k] / sum * scale;
 }
 
 // The same choice with one warp per token (up to 256 router outputs: eight per lane, in registers): the softmax's
@@ -162,7 +165,7 @@ moe_topk_kernel(float* __restrict__ logits, int n_tokens, int E, int top, int mo
 #define MT_PER_LANE 8
 __global__ void __launch_bounds__(128)
 moe_topk_warp_kernel(const float* __restrict__ logits, int n_tokens, int E, int top, int mode,
-                     const float* __restrict__ corr, int* __restrict__ idx, float* __restrict__ wt) {
+                     const float* __restrict__ corr, int* __restrict__ idx, float* __restrict__ wt, float scale) {
   pdl_launch_dependents();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -211,16 +214,17 @@ moe_topk_warp_kernel(const float* __restrict__ logits, int n_tokens, int E, int 
     for (int j = 0; j < MT_PER_LANE; j++)
       if (lane + 32 * j == be) c[j] = -INFINITY;
     if (k == 0) first = bz;
-    // mode 0: the first chosen is the largest logit; mode 2: the chosen logit's own sigmoid
-    const float w = mode == 1 ? bz : mode == 2 ? 1.0f / (1.0f + expf(-bz)) : expf(bz - first);
+    // mode 0: the first chosen is the largest logit; modes 2 and 3: the chosen logit's own sigmoid
+    const float w = mode == 1 ? bz : mode >= 2 ? 1.0f / (1.0f + expf(-bz)) : expf(bz - first);
     sum += w;
     if (lane == (k & 31)) {
       idx[(size_t)t * top + k] = be;
-      if (mode != 0) wt[(size_t)t * top + k] = w;
+      if (mode == 1 || mode == 2) wt[(size_t)t * top + k] = w * scale;
       else chosen = w;                          // top <= 32: one round per lane
     }
   }
-  if (mode == 0 && lane < top) wt[(size_t)t * top + lane] = chosen / sum;
+  if (mode == 0 && lane < top) wt[(size_t)t * top + lane] = chosen / sum * scale;
+  if (mode == 3 && lane < top) wt[(size_t)t * top + lane] = chosen * (scale / (sum + 1e-20f));
 }
 
 // ----------------------------------------------------------------------------- sort
@@ -560,21 +564,21 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place, c
 // ----------------------------------------------------------------------------- launchers
 // The choice alone, from float32 logits [T, E] that a product left (the thread-per-token form overwrites them).
 extern "C" int qd_moe_topk(float* logits, int T, int E, int top, int mode, const float* corr, int* idx, float* wt,
-                           cudaStream_t stream) {
+                           float scale, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (top < 1 || top > E || top > MOE_MAX_TOP) return QD_ERR_UNSUPPORTED;
+  if (mode < 0 || mode > 3 || top < 1 || top > E || top > MOE_MAX_TOP) return QD_ERR_UNSUPPORTED;
   if (E <= 32 * MT_PER_LANE)
     qd_launch(moe_topk_warp_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, (const float*)logits, T, E, top, mode, corr,
-              idx, wt);
+              idx, wt, scale);
   else
-    qd_launch(moe_topk_kernel, dim3((T + 127) / 128), dim3(128), 0, stream, logits, T, E, top, mode, corr, idx, wt);
+    qd_launch(moe_topk_kernel, dim3((T + 127) / 128), dim3(128), 0, stream, logits, T, E, top, mode, corr, idx, wt, scale);
   return qd_last_error();
 }
 
 // logits: float32 scratch [T, E] (left with the chosen entries at -inf)
 extern "C" int qd_moe_route(const void* h, const void* wr, const float* br, const void* wsg, int dtype, int T, int D,
                             int E, int top, int mode, const float* corr, float* logits, int* idx, float* wt,
-                            float* sgate, cudaStream_t stream) {
+                            float* sgate, float scale, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (top < 1 || top > E || top > MOE_MAX_TOP) return QD_ERR_UNSUPPORTED;
   const int rows = E + (wsg ? 1 : 0);
@@ -588,7 +592,7 @@ extern "C" int qd_moe_route(const void* h, const void* wr, const float* br, cons
   else if (dtype == QD_BF16) { if (al && D % 8 == 0) MR_GO(bf16, true); else MR_GO(bf16, false); }
   else return QD_ERR_UNSUPPORTED;
 #undef MR_GO
-  return qd_moe_topk(logits, T, E, top, mode, corr, idx, wt, stream);
+  return qd_moe_topk(logits, T, E, top, mode, corr, idx, wt, scale, stream);
 }
 
 extern "C" int qd_moe_sort(const int* idx, int n_pairs, int E, int E_real, int tile_rows, int max_tiles, int* place,

@@ -228,6 +228,12 @@ extern "C" int qd_add_tanh_norm(float* x, int T, int D,
 }
 
 // ------------------------------------------------------------------------------------------------ gated activation
+__device__ __forceinline__ float gated_one(float g, float u, int kind, float limit, float alpha) {
+  if (kind != 1) return qd_gated(g, u, kind);         // QD_ACT_SILU, QD_ACT_GELU_TANH
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
 __global__ void __launch_bounds__(256)
 gated_act_kernel(const void* __restrict__ gu, int in_dtype, void* __restrict__ out, int out_dtype, int F, size_t n,
                  int kind, float limit, float alpha) {
@@ -235,25 +241,12 @@ gated_act_kernel(const void* __restrict__ gu, int in_dtype, void* __restrict__ o
   pdl_wait();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
     const size_t t = i / F, f = i - t * F;
-    float g = ld_code(gu, in_dtype, t * 2 * F + f), u = ld_code(gu, in_dtype, t * 2 * F + F + f);
-    float v;
-    if (kind == 0) v = g / (1.0f + expf(-g)) * u;
-    else {
-      g = fminf(g, limit);
-      u = fminf(fmaxf(u, -limit), limit);
-      v = g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
-    }
-    st_code(out, out_dtype, i, v);
+    const float g = ld_code(gu, in_dtype, t * 2 * F + f), u = ld_code(gu, in_dtype, t * 2 * F + F + f);
+    st_code(out, out_dtype, i, gated_one(g, u, kind, limit, alpha));
   }
 }
 
 // Four elements per thread with 16-byte (float32) or 8-byte (bfloat16) accesses: F a multiple of 4, aligned pointers.
-__device__ __forceinline__ float gated_one(float g, float u, int kind, float limit, float alpha) {
-  if (kind == 0) return g / (1.0f + expf(-g)) * u;
-  g = fminf(g, limit);
-  u = fminf(fmaxf(u, -limit), limit);
-  return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
-}
 __global__ void __launch_bounds__(256)
 gated_act_vec_kernel(const void* __restrict__ gu, int in_dtype, void* __restrict__ out, int out_dtype, int F4, size_t n4,
                      int kind, float limit, float alpha) {
@@ -306,5 +299,29 @@ extern "C" int qd_token_gate(const void* z, int z_dtype, const void* table, int 
   unsigned blocks = (unsigned)((n + 255) / 256 < 65535 ? (n + 255) / 256 : 65535);
   qd_launch(token_gate_kernel, dim3(blocks), dim3(256), 0, stream, z, z_dtype, table, table_dtype, tokens, out,
             out_dtype, W, n);
+  return qd_last_error();
+}
+
+// ------------------------------------------------------------------------------------------------ soft cap
+// z <- cap * tanh(z / cap), element by element, in place.  Four elements a thread.
+__global__ void __launch_bounds__(256)
+soft_cap_kernel(float* __restrict__ z, size_t n, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  const float inv = 1.0f / cap;
+  if (i + 4 <= n) {
+    float4 v = *reinterpret_cast<float4*>(z + i);
+    v = make_float4(cap * tanhf(v.x * inv), cap * tanhf(v.y * inv), cap * tanhf(v.z * inv), cap * tanhf(v.w * inv));
+    *reinterpret_cast<float4*>(z + i) = v;
+    return;
+  }
+  for (size_t j = i; j < n; j++) z[j] = cap * tanhf(z[j] * inv);
+}
+
+extern "C" int qd_soft_cap(float* z, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.0f) || ((uintptr_t)z & 15)) return QD_ERR_UNSUPPORTED;
+  qd_launch(soft_cap_kernel, dim3((unsigned)((n + 1023) / 1024)), dim3(256), 0, stream, z, (size_t)n, cap);
   return qd_last_error();
 }

@@ -12,6 +12,7 @@
 //   write     q to a dense [T, H*d] tensor, k and v to the token's slot of the paged cache
 //             (a page: keys [G, page_size, d], then values [G, page_size, vd])
 //
+// G = 0: the row holds queries alone (a layer that attends over another layer's keys and values).
 // Everything is float32 until the stores.  The order of every sum depends on the sizes only.
 #include "common.cuh"
 #include "short_conv.cuh"
@@ -68,7 +69,7 @@ qkv_prep_kernel(QkvPrep a) {
   float fq = 1.f, fk = 1.f;
   if (a.norm_mode == 1) {
     fq = 1.0f / sqrtf(block_sum(ssq, scratch) / (float)nq + a.eps);
-    fk = 1.0f / sqrtf(block_sum(ssk, scratch) / (float)nk + a.eps);
+    if (G) fk = 1.0f / sqrtf(block_sum(ssk, scratch) / (float)nk + a.eps);
   }
   __syncthreads();
   // every request brings one token: channel c's kept inputs were read by this thread alone, which now moves them on
@@ -170,9 +171,9 @@ extern "C" int qd_qkv_prep(const float* u, long long ld, int T, int n_requests, 
                            cudaStream_t stream) {
   if (T <= 0) return 0;
   const long long C = (long long)H * d + (long long)G * d + (long long)G * vd;
-  if (d <= 0 || d > QP_MAX_D || vd <= 0 || G <= 0 || H <= 0 || rotary_dim < 0 || rotary_dim > d ||
+  if (d <= 0 || d > QP_MAX_D || vd <= 0 || G < 0 || (G == 0 && write_kv) || H <= 0 || rotary_dim < 0 || rotary_dim > d ||
       (rotary_dim & 1) || taps < 0 || (taps > 1 && !state) || (taps > 0 && !conv_w) || norm_mode < 0 || norm_mode > 2 ||
-      (norm_mode == 1 && (!wq || !wk)) || (rotary_dim > 0 && (!cos_t || !sin_t)) || n_requests > 65535)
+      (norm_mode == 1 && (!wq || (G && !wk))) || (rotary_dim > 0 && (!cos_t || !sin_t)) || n_requests > 65535)
     return QD_ERR_UNSUPPORTED;
   const size_t smem = ((size_t)C + 40) * sizeof(float);
   if (smem > 200 * 1024) return QD_ERR_UNSUPPORTED;

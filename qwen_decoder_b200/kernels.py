@@ -219,25 +219,31 @@ def elementwise_plain_next() -> None:
     fn()
 
 
-def swiglu_partial(part: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:
+# gated activations by code: silu(g) * u; the clamped gate (see ``gated_act``); gelu(g) * u in its tanh form
+ACT_SILU, ACT_CLAMPED, ACT_GATED_GELU = 0, 1, 2
+
+
+def swiglu_partial(part: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                   act: int = ACT_SILU) -> None:
     """out[t, f] = silu(sum_p part[p, t, f]) * (sum_p part[p, t, F + f]) from the float32 partial sums
-    [n_parts, T, 2F] of a split-K gate/up product (plus ``bias`` float32 [2F], if given); out bfloat16."""
+    [n_parts, T, 2F] of a split-K gate/up product (plus ``bias`` float32 [2F], if given); out bfloat16.  ``act``:
+    ``ACT_SILU``, or ``ACT_GATED_GELU`` in silu's place (so in every fused form of the gate)."""
     T, F = out.shape
     assert part.dim() == 3 and tuple(part.shape[1:]) == (T, 2 * F) and part.dtype == torch.float32
     assert out.dtype == torch.bfloat16 and F % 4 == 0
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == 2 * F and bias.is_contiguous())
     _contig(part, "part"); _contig(out, "out")
-    _check(library("elementwise").qd_swiglu_partial(_ptr(part), _I(part.shape[0]), _ptr(bias), _ptr(out), _I(T), _I(F), _stream()),
-           "swiglu_partial")
+    _check(library("elementwise").qd_swiglu_partial(_ptr(part), _I(part.shape[0]), _ptr(bias), _ptr(out), _I(T), _I(F),
+                                                    _I(act), _stream()), "swiglu_partial")
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t, f] = silu(gate_up[t, f]) * gate_up[t, F + f]."""
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, act: int = ACT_SILU) -> None:
+    """out[t, f] = act(gate_up[t, f]) * gate_up[t, F + f]."""
     T, F = out.shape
     assert gate_up.shape == (T, 2 * F) and gate_up.dtype == out.dtype
     _contig(gate_up, "gate_up"); _contig(out, "out")
-    _check(library("elementwise").qd_swiglu(_ptr(gate_up), _ptr(out), _I(dtype_code(out.dtype)), _I(T),
-                                            _I(F), _stream()), "swiglu")
+    _check(library("elementwise").qd_gate_mul(_ptr(gate_up), _ptr(out), _I(dtype_code(out.dtype)), _I(T),
+                                              _I(F), _I(act), _stream()), "swiglu")
 
 
 # ------------------------------------------------------------------------ gemm
@@ -268,7 +274,7 @@ STREAM_RESIDENT_TOKENS = 16    # from there up to here it still takes a product 
 STREAM_RESIDENT_MAX_SHARES = 32
 TC5_POLICY_TOKENS = 16         # from SKINNY_POLICY_TOKENS up to here the tcgen05 kernel; 16 = never:
 # on row-major weights it reads 128-byte pieces of 128 rows per copy and stays below the library product
-EPI_STORE, EPI_PARTIAL, EPI_SWIGLU = 0, 1, 2
+EPI_STORE, EPI_PARTIAL, EPI_SWIGLU = 0, 1, 2      # EPI_SWIGLU + 256 * act: another gated activation in silu's place
 
 
 def few_token_impl(T: int) -> str:
@@ -463,15 +469,15 @@ def gemm_skinny_partial(x: torch.Tensor, w: torch.Tensor, splits: int) -> torch.
 
 
 def gemm_skinny_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor,
-                       bias: Optional[torch.Tensor] = None) -> None:
-    """out[T, F] = silu(x @ Wg^T) * (x @ Wu^T) with w_gate_up = [Wg; Wu] of shape [2F, K]; ``bias`` float32 [2F]: added
+                       bias: Optional[torch.Tensor] = None, act: int = ACT_SILU) -> None:
+    """out[T, F] = act(x @ Wg^T) * (x @ Wu^T) with w_gate_up = [Wg; Wu] of shape [2F, K]; ``bias`` float32 [2F]: added
     to both products first."""
     T, K = x.shape
     N = w_gate_up.shape[0]
     assert skinny_supported(x, w_gate_up, 1 << 30) and out.shape == (T, N // 2) and out.dtype == torch.bfloat16
     _contig(w_gate_up, "w"); _contig(out, "out")
     assert bias is None or (bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous())
-    _skinny_call(x, w_gate_up, bias, out, None, T, N, K, 1, EPI_SWIGLU, "gemm_skinny_swiglu")
+    _skinny_call(x, w_gate_up, bias, out, None, T, N, K, 1, EPI_SWIGLU + 256 * act, "gemm_skinny_swiglu")
 
 
 def ffn_stream_supported(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor) -> bool:
@@ -487,8 +493,9 @@ FFN_SYNC_WORDS = 64      # words of device memory a layer's one-launch feed-forw
 
 
 def ffn_stream(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, barrier: torch.Tensor,
-               timeline: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """float32 partial sums [splits, T, D] of (silu(x Wg^T) * (x Wu^T)) Wd^T (``bias`` float32 [2F], if given, joins both
+               timeline: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
+               act: int = ACT_SILU) -> torch.Tensor:
+    """float32 partial sums [splits, T, D] of (act(x Wg^T) * (x Wu^T)) Wd^T (``bias`` float32 [2F], if given, joins both
     products of x) for up to 8 tokens, in one
     launch of the weight streamer: between the two products a CTA waits for the others' columns of h that its
     share of the second product reads, its producer warp meanwhile fetches the second product's first weights.  ``barrier``: ``FFN_SYNC_WORDS`` int32 words
@@ -505,7 +512,7 @@ def ffn_stream(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, b
     part = torch.empty((splits, T, D), dtype=torch.float32, device=x.device)
     _check(library("gemm_stream").qd_ffn_stream(
         _ptr(w_gate_up), _ptr(bias), _ptr(x), _LL(x.stride(0)), _ptr(h), _LL(h.stride(0)), _ptr(w_down), _ptr(part), _I(T), _I(D),
-        _I(F), _I(splits), _ptr(barrier), _I(stream_max_ctas()), _ptr(timeline), _stream()), "ffn_stream")
+        _I(F), _I(splits), _ptr(barrier), _I(stream_max_ctas()), _I(act), _ptr(timeline), _stream()), "ffn_stream")
     return part
 
 
@@ -710,11 +717,11 @@ LATENT_MAX_RANK = 512
 def latent_prep(u: torch.Tensor, q_off: int, q_rank: int, kv_off: int, r: int, dr: int, wq_norm: torch.Tensor,
                 wkv_norm: torch.Tensor, eps: float, cos: torch.Tensor, sin: torch.Tensor, rot_dims: int,
                 positions: torch.Tensor, slot_map: torch.Tensor, cq: torch.Tensor, cache: torch.Tensor,
-                write_cache: bool) -> None:
+                write_cache: bool, pairing: int = 0) -> None:
     """From the float32 projections u [T, *]: cq [T, q_rank] = RMS norm of the query latent times its weight, and
     the cache row [normed latent (r) | rotated key part (dr)] written to each token's slot of ``cache``
     [pages, page_size, r + dr].  Norms and rotation in float32; ``rot_dims`` leading elements of the key part turn,
-    pairs (2i, 2i + 1).  ``q_rank`` 0: there is no query latent (``cq`` is empty, ``wq_norm`` unused)."""
+    pairs (2i, 2i + 1), or (i, i + rot_dims / 2) with ``pairing`` 1.  ``q_rank`` 0: there is no query latent (``cq`` is empty, ``wq_norm`` unused)."""
     T = u.shape[0]
     assert u.dtype == torch.float32 and u.stride(1) == 1 and cq.shape == (T, q_rank) and cq.dtype == cache.dtype
     assert cache.shape[-1] == r + dr and wq_norm.dtype == wkv_norm.dtype == torch.float32
@@ -723,12 +730,12 @@ def latent_prep(u: torch.Tensor, q_off: int, q_rank: int, kv_off: int, r: int, d
     _check(library("latent_attention").qd_latent_prep(
         _ptr(u), _LL(u.stride(0)), _I(q_off), _I(q_rank), _I(kv_off), _I(r), _I(dr), _ptr(wq_norm), _ptr(wkv_norm),
         _F(eps), _ptr(cos), _ptr(sin), _I(rot_dims), _ptr(positions), _ptr(slot_map), _ptr(cq), _ptr(cache),
-        _I(dtype_code(cache.dtype)), _I(1 if write_cache else 0), _I(T), _stream()), "latent_prep")
+        _I(dtype_code(cache.dtype)), _I(1 if write_cache else 0), _I(T), _I(pairing), _stream()), "latent_prep")
 
 
 def latent_absorb(q: torch.Tensor, wuk: torch.Tensor, qcat: torch.Tensor, H: int, dn: int, dr: int, r: int,
                   cos: torch.Tensor, sin: torch.Tensor, rot_dims: int, positions: torch.Tensor,
-                  pre: Optional[torch.Tensor] = None) -> None:
+                  pre: Optional[torch.Tensor] = None, pairing: int = 0) -> None:
     """qcat[t, h] = [Wuk_h^T q_unrotated[t, h] (r) | rotate(q_rotated[t, h]) (dr)], float32; q float32
     [T, H * (dn + dr)], wuk [H * dn, r].  ``pre`` (float32 [H, T, r]): the first part, already made by a batched
     library product."""
@@ -739,7 +746,7 @@ def latent_absorb(q: torch.Tensor, wuk: torch.Tensor, qcat: torch.Tensor, H: int
     _contig(wuk, "wuk"); _contig(qcat, "qcat")
     _check(library("latent_attention").qd_latent_absorb(
         _ptr(q), _LL(q.stride(0)), _ptr(wuk), _I(dtype_code(wuk.dtype)), _ptr(qcat), _I(T), _I(H), _I(dn), _I(dr), _I(r), _ptr(cos),
-        _ptr(sin), _I(rot_dims), _ptr(positions), _ptr(pre), _stream()), "latent_absorb")
+        _ptr(sin), _I(rot_dims), _ptr(positions), _ptr(pre), _I(pairing), _stream()), "latent_absorb")
 
 
 def latent_attend(qcat: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, token_req: torch.Tensor,
@@ -847,9 +854,8 @@ def mamba_gate_norm(y: torch.Tensor, u: torch.Tensor, z_off: int, w: torch.Tenso
 
 
 # ------------------------------------------------------------------ routed experts
-ACT_SILU, ACT_CLAMPED = 0, 1     # gated activations: silu(g) * u; the clamped gate (see ``gated_act``)
 MOE_MAX_TOP = 32
-MOE_ROUTE_TOP_SOFTMAX, MOE_ROUTE_SOFTMAX_ALL, MOE_ROUTE_TOP_SIGMOID = 0, 1, 2
+MOE_ROUTE_TOP_SOFTMAX, MOE_ROUTE_SOFTMAX_ALL, MOE_ROUTE_TOP_SIGMOID, MOE_ROUTE_TOP_SIGMOID_NORM = 0, 1, 2, 3
 MOE_FEW_ROWS = 8          # rows of one expert that the weight-streaming grouped product takes as one tile
 
 
@@ -866,11 +872,12 @@ def moe_tile_rows(n_pairs: int, E: int, K1: int, K2: int, dtype: torch.dtype) ->
 
 def moe_route(h: torch.Tensor, wr: torch.Tensor, br: Optional[torch.Tensor], wsg: Optional[torch.Tensor], top: int,
               idx: torch.Tensor, wt: torch.Tensor, sgate: Optional[torch.Tensor], mode: int = MOE_ROUTE_TOP_SOFTMAX,
-              correction: Optional[torch.Tensor] = None) -> None:
+              correction: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
     """idx, wt [T, top] from the float32 logits wr h (+ br).  ``MOE_ROUTE_TOP_SOFTMAX``: the ``top`` largest logits and
     the softmax over those.  ``MOE_ROUTE_SOFTMAX_ALL``: scores = softmax over all outputs; the ``top`` largest of
     score + correction are chosen and weigh by their plain scores.  ``MOE_ROUTE_TOP_SIGMOID``: the ``top`` largest
-    logits, each weighed by its own sigmoid.  sgate[t] = sigmoid(wsg . h[t]) when a shared expert's gate vector is
+    logits, each weighed by its own sigmoid; ``MOE_ROUTE_TOP_SIGMOID_NORM`` divides those by their sum (+ 1e-20).  All
+    weights are multiplied by ``scale``.  sgate[t] = sigmoid(wsg . h[t]) when a shared expert's gate vector is
     given."""
     T, D = h.shape
     E = wr.shape[0]
@@ -882,13 +889,13 @@ def moe_route(h: torch.Tensor, wr: torch.Tensor, br: Optional[torch.Tensor], wsg
     logits = torch.empty((T, E), dtype=torch.float32, device=h.device)
     _check(library("moe").qd_moe_route(_ptr(h), _ptr(wr), _ptr(br), _ptr(wsg), _I(dtype_code(h.dtype)), _I(T), _I(D),
                                        _I(E), _I(top), _I(mode), _ptr(correction), _ptr(logits), _ptr(idx), _ptr(wt),
-                                       _ptr(sgate), _stream()),
+                                       _ptr(sgate), _F(scale), _stream()),
            "moe_route")
     _launch_count[0] += 1
 
 
 def moe_choose(logits: torch.Tensor, top: int, idx: torch.Tensor, wt: torch.Tensor, mode: int = MOE_ROUTE_TOP_SOFTMAX,
-               correction: Optional[torch.Tensor] = None) -> None:
+               correction: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
     """The choice of ``moe_route`` from float32 logits [T, E] that a product left (they may be overwritten)."""
     T, E = logits.shape
     assert logits.dtype == torch.float32 and idx.dtype == torch.int32 and wt.dtype == torch.float32
@@ -896,7 +903,7 @@ def moe_choose(logits: torch.Tensor, top: int, idx: torch.Tensor, wt: torch.Tens
     assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
     _contig(logits, "logits")
     _check(library("moe").qd_moe_topk(_ptr(logits), _I(T), _I(E), _I(top), _I(mode), _ptr(correction), _ptr(idx),
-                                      _ptr(wt), _stream()), "moe_choose")
+                                      _ptr(wt), _F(scale), _stream()), "moe_choose")
 
 
 def moe_sort(idx: torch.Tensor, E: int, tile_rows: int, max_tiles: int, place: torch.Tensor, pair_at: torch.Tensor,
@@ -1205,13 +1212,21 @@ def add_tanh_norm(x: torch.Tensor, addends, norms, rows: Optional[torch.Tensor] 
 def gated_act(gate_up: torch.Tensor, out: torch.Tensor, act: int = ACT_SILU, limit: float = 0.0,
               alpha: float = 1.0) -> None:
     """out[t, f] = act(g, u), g = gate_up[t, f], u = gate_up[t, F + f].  ``ACT_SILU``: silu(g) * u.  ``ACT_CLAMPED``:
-    g' = min(g, limit), u' = clamp(u, -limit, limit), g' * sigmoid(alpha * g') * (u' + 1)."""
+    g' = min(g, limit), u' = clamp(u, -limit, limit), g' * sigmoid(alpha * g') * (u' + 1).  ``ACT_GATED_GELU``:
+    0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))) * u."""
     T, F = out.shape
     assert gate_up.shape == (T, 2 * F)
     _contig(gate_up, "gate_up"); _contig(out, "out")
     _check(library("norm_act").qd_gated_act(_ptr(gate_up), _I(dtype_code(gate_up.dtype)), _ptr(out),
                                             _I(dtype_code(out.dtype)), _I(T), _I(F), _I(act), _F(limit), _F(alpha),
                                             _stream()), "gated_act")
+
+
+def soft_cap(z: torch.Tensor, cap: float) -> None:
+    """z <- cap * tanh(z / cap), float32, in place."""
+    assert z.dtype == torch.float32
+    _contig(z, "z")
+    _check(library("norm_act").qd_soft_cap(_ptr(z), _LL(z.numel()), _F(cap), _stream()), "soft_cap")
 
 
 def token_gate(z: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor) -> None:
@@ -1258,13 +1273,14 @@ def qk_norm_rope_write(qkv: torch.Tensor, H: int, G: int, d: int, vd: int, wq: O
 def sink_attention_generic(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, block_table: torch.Tensor,
                            token_req: torch.Tensor, positions: torch.Tensor, H: int, G: int, d: int, vd: int,
                            page_size: int, scale: float, window: int, sinks: Optional[torch.Tensor], chunk: int = 0,
-                           gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, gate_elem: bool = False) -> None:
+                           gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, gate_elem: bool = False,
+                           cap: float = 0.0) -> None:
     """Attention of every token over keys 0..pos (or the last ``window``; with ``chunk`` only those of the query's
     own block of ``chunk`` positions) of its request with a sink in the softmax's denominator (``sinks`` float32 [H],
     or None), values of size ``vd``; q [T, H*d], out [T, H*vd] (rows may be strided: a column range of a wider
     tensor); head h's output is multiplied by ``out_scale`` and, with ``gate`` (float32 [T, >= H] logits, rows may be
     strided), by sigmoid(gate[t, h]) or, with ``gate_elem`` (gate [T, >= H*vd]), element by element by
-    sigmoid(gate[t, h*vd + i]); float32 arithmetic, any sizes."""
+    sigmoid(gate[t, h*vd + i]); ``cap`` > 0: a score s counts as cap * tanh(s / cap); float32 arithmetic, any sizes."""
     T = q.shape[0]
     assert q.shape == (T, H * d) and out.shape == (T, H * vd) and q.dtype == out.dtype == kv.dtype
     assert q.stride(1) == 1 and out.stride(1) == 1
@@ -1278,7 +1294,7 @@ def sink_attention_generic(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor,
         _ptr(q), _LL(q.stride(0)), _ptr(out), _LL(out.stride(0)), _ptr(kv), _I(dtype_code(q.dtype)), _ptr(block_table),
         _I(block_table.shape[1]), _ptr(token_req), _ptr(positions), _I(T), _I(H), _I(G), _I(d), _I(vd), _I(page_size),
         _F(scale), _I(window), _ptr(sinks), _I(chunk), _ptr(gate), _LL(gate.stride(0) if gate is not None else 0),
-        _I(1 if gate_elem else 0), _F(out_scale), _stream()), "sink_attention_generic")
+        _I(1 if gate_elem else 0), _F(out_scale), _F(cap), _stream()), "sink_attention_generic")
 
 
 SINK_MMA_ROWS = 64       # rows, (token, head within the group) pairs, of one tile of the tensor-core kernel
@@ -1295,11 +1311,11 @@ def sink_attention_mma(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, blo
                        cu_tokens: torch.Tensor, start_pos: torch.Tensor, n_requests: int, n_tokens: int, H: int, G: int,
                        d: int, vd: int, page_size: int, scale: float, window: int, sinks: Optional[torch.Tensor],
                        splits: int = 1, chunk: int = 0, gate: Optional[torch.Tensor] = None,
-                       out_scale: float = 1.0, gate_elem: bool = False) -> None:
+                       out_scale: float = 1.0, gate_elem: bool = False, cap: float = 0.0) -> None:
     """``sink_attention_generic`` on tensor cores for portions of ``n_requests`` requests (rows cu_tokens[r] ..
     cu_tokens[r+1]-1 of q and out, at positions start_pos[r]..): a decoded token is a portion of one.  ``splits`` > 1
     shares every tile's keys among that many CTAs (for steps of few tokens over long contexts).  ``chunk``, ``gate``,
-    ``gate_elem``, ``out_scale`` and strided rows of ``out`` as for the generic kernel."""
+    ``gate_elem``, ``out_scale``, ``cap`` and strided rows of ``out`` as for the generic kernel."""
     assert q.dtype == out.dtype == kv.dtype == torch.bfloat16 and q.shape[1] == H * d and out.shape[1] == H * vd
     assert out.stride(1) == 1 and out.stride(0) % 2 == 0
     assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
@@ -1325,7 +1341,7 @@ def sink_attention_mma(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, blo
         _I(n_requests), _I(n_tokens), _I(tiles), _I(H), _I(G), _I(d), _I(vd), _I(page_size), _F(scale), _I(window),
         _ptr(sinks), _I(splits), _ptr(part_o), _ptr(part_ml), _ptr(tickets), _I(chunk), _ptr(gate),
         _LL(gate.stride(0) if gate is not None else 0), _I(1 if gate_elem else 0), _F(out_scale), _LL(out.stride(0)),
-        _stream()),
+        _F(cap), _stream()),
         "sink_attention_mma")
     if splits > 1 and tickets is None:
         _launch_count[0] += 1
@@ -1346,9 +1362,11 @@ def qkv_prep(u: torch.Tensor, H: int, G: int, d: int, vd: int, conv_w: Optional[
     mean square over the whole projection times wq [H*d] / wk [G*d], before the rotation; "head": every head divided
     by its own, without weights, after the rotation when ``norm_after``; the first ``rotary_dim`` elements of every
     head of q and k turned by the table rows of ``ctx.positions``; q to q_out [T, H*d], k and v to the token's slot of
-    ``kv`` (pages of [G, page_size, d] keys then [G, page_size, vd] values)."""
+    ``kv`` (pages of [G, page_size, d] keys then [G, page_size, vd] values).  ``G`` = 0: u holds queries alone (and
+    nothing is written to the cache)."""
     T = u.shape[0]
     C = H * d + G * d + G * vd
+    assert G > 0 or not write_kv
     assert u.dtype == torch.float32 and u.shape[1] >= C and u.stride(1) == 1
     assert q_out.shape == (T, H * d) and q_out.is_contiguous()
     taps = 0
@@ -1357,7 +1375,8 @@ def qkv_prep(u: torch.Tensor, H: int, G: int, d: int, vd: int, conv_w: Optional[
         assert conv_w.shape == (C, taps) and conv_w.dtype == torch.float32 and conv_w.is_contiguous()
         assert taps == 1 or (state is not None and state.dtype == torch.float32 and state.is_contiguous())
     if norm == "whole":
-        assert wq.dtype == wk.dtype == torch.float32 and wq.numel() == H * d and wk.numel() == G * d
+        assert wq.dtype == torch.float32 and wq.numel() == H * d
+        assert G == 0 or (wk.dtype == torch.float32 and wk.numel() == G * d)
     if rotary_dim:
         assert cos.dtype == sin.dtype == torch.float32 and cos.shape[1] == rotary_dim // 2
     if write_kv:
@@ -1449,14 +1468,16 @@ def linear_pad(d: int) -> int:
 def linear_prep(u: torch.Tensor, H: int, G: int, d: int, dv: int, conv_w: Optional[torch.Tensor],
                 state: Optional[torch.Tensor], conv_off: int, ctx, update_state: bool, unit_eps: Optional[float],
                 rotary_dim: int, pairing: int, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], q_scale: float,
-                k_scale: float, b_off: int, a_off: int, A_log: Optional[torch.Tensor], dt_bias: Optional[torch.Tensor]):
+                k_scale: float, b_off: int, a_off: int, A_log: Optional[torch.Tensor], dt_bias: Optional[torch.Tensor],
+                k_mul: Optional[torch.Tensor] = None):
     """From the float32 sums u [T, >= 2*G*d + H*dv] (q | k | v | ...; rows may be strided): (q, k, v, beta, g) for
     ``linear_scan``.  With ``conv_w`` (float32 [2*G*d + H*dv, taps]) every channel of q, k and v passes a causal
     convolution (the last taps - 1 inputs of a request live at ``conv_off`` of its row of ``state`` and are moved on
     when ``update_state``) and silu; else v is a view of u.  ``unit_eps``: q and k of every head divided by
     sqrt(sum of squares + unit_eps).  The first ``rotary_dim`` elements of a head turn by the table rows of
     ``ctx.positions``; then q times ``q_scale``, k times ``k_scale``.  ``b_off`` / ``a_off`` >= 0: the columns of u whose
-    sigmoid is beta, and g = exp(-exp(A_log) softplus(u + dt_bias)); None otherwise."""
+    sigmoid is beta, and g = exp(-exp(A_log) softplus(u + dt_bias)); None otherwise.  ``k_mul`` float32 [T, G]: multiplies
+    k's heads as well."""
     T = u.shape[0]
     C = 2 * G * d + H * dv
     assert u.dtype == torch.float32 and u.stride(1) == 1 and u.shape[1] >= max(C, b_off + H, a_off + H)
@@ -1469,6 +1490,7 @@ def linear_prep(u: torch.Tensor, H: int, G: int, d: int, dv: int, conv_w: Option
         assert cos.dtype == sin.dtype == torch.float32 and cos.shape[1] == rotary_dim // 2
     if a_off >= 0:
         assert A_log.dtype == dt_bias.dtype == torch.float32 and A_log.numel() == dt_bias.numel() == H
+    assert k_mul is None or (k_mul.shape == (T, G) and k_mul.dtype == torch.float32 and k_mul.is_contiguous())
     DP = linear_pad(d)
     new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=u.device)
     q, k = new(T, G, DP), new(T, G, DP)
@@ -1480,38 +1502,95 @@ def linear_prep(u: torch.Tensor, H: int, G: int, d: int, dv: int, conv_w: Option
         _ptr(state if taps > 1 else None), _LL(state.stride(0) if state is not None else 0), _LL(conv_off),
         _ptr(ctx.token_request), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _I(1 if update_state else 0),
         _I(0 if unit_eps is None else 1), _F(unit_eps or 0.0), _I(rotary_dim), _I(pairing), _ptr(cos), _ptr(sin),
-        _ptr(ctx.positions), _F(q_scale), _F(k_scale), _I(b_off), _I(a_off), _ptr(A_log), _ptr(dt_bias), _ptr(q), _ptr(k),
+        _ptr(ctx.positions), _F(q_scale), _F(k_scale), _I(b_off), _I(a_off), _ptr(A_log), _ptr(dt_bias), _ptr(k_mul), _ptr(q), _ptr(k),
         _ptr(v if taps else None), _ptr(beta), _ptr(g), _stream()), "linear_prep")
     if update_state and taps > 1 and T != ctx.num_requests:
         _launch_count[0] += 1
     return q, k, v, beta, g
 
 
-def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: Optional[torch.Tensor], H: int,
-                d: int, dv: int, state: torch.Tensor, s_off: int, ctx, write_state: bool, gate: torch.Tensor,
-                norm: Optional[torch.Tensor], eps: float, out_scale: float, out: torch.Tensor) -> None:
+class ExpGates:
+    """What a head with exponential gates needs: the stacked product's float32 sums ``u`` [T, *] with the gates' logits at
+    columns ``i_off`` and ``f_off``, their biases (float32 [H]), the cap, and where the heads' running maxima are in a state row."""
+
+    def __init__(self, u, i_off, f_off, i_bias, f_bias, cap, m_off):
+        assert u.dtype == torch.float32 and u.stride(1) == 1 and i_bias.dtype == f_bias.dtype == torch.float32
+        self.u, self.i_off, self.f_off, self.i_bias, self.f_bias = u, int(i_off), int(f_off), i_bias, f_bias
+        self.cap, self.m_off = float(cap), int(m_off)
+
+
+def linear_exp_gates(e: ExpGates, H: int, state: torch.Tensor, ctx, write_state: bool):
+    """(g, in, low) float32 [T, H] of portions: with i = cap tanh((u_i + ib) / cap), f = logsigmoid(cap tanh((u_f + fb) / cap))
+    and m' = max(f + m, i) token by token from the requests' kept maxima, g = exp(f + m - m'), in = exp(i - m'),
+    low = exp(-m'); the last maxima go back to the state rows when ``write_state``."""
+    T = e.u.shape[0]
+    assert state.dtype == torch.float32 and e.m_off + H <= state.shape[1] and max(e.i_off, e.f_off) + H <= e.u.shape[1]
+    _contig(state, "state")
+    g, inn, low = (torch.empty((T, H), dtype=torch.float32, device=e.u.device) for _ in range(3))
+    _check(library("linear_scan").qd_linear_exp_gates(
+        _ptr(e.u), _LL(e.u.stride(0)), _I(e.i_off), _I(e.f_off), _ptr(e.i_bias), _ptr(e.f_bias), _F(e.cap), _I(T),
+        _I(ctx.num_requests), _I(H), _ptr(state), _LL(state.stride(0)), _LL(e.m_off), _ptr(ctx.cu_tokens), _ptr(ctx.state_slots),
+        _I(1 if write_state else 0), _ptr(g), _ptr(inn), _ptr(low), _stream()), "linear_exp_gates")
+    return g, inn, low
+
+
+def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: Optional[torch.Tensor], beta: Optional[torch.Tensor],
+                H: int, d: int, dv: int, state: torch.Tensor, s_off: int, ctx, write_state: bool, gate: torch.Tensor,
+                norm: Optional[torch.Tensor], eps: float, out_scale: float, out: torch.Tensor, gate_kind: int = 0,
+                exp_gates: Optional[ExpGates] = None, low: Optional[torch.Tensor] = None, q_scale: float = 1.0,
+                k_scale: float = 1.0) -> None:
     """Per (request, head), token by token: S <- g S;  x = v, or with ``beta`` (the delta rule) beta (v - S^T k);
-    S <- S + k x^T;  o = S^T q;  out[t, head] = o / sqrt(mean(o^2) + eps) * norm * silu(gate) * out_scale.  q, k float32
-    [T, G, linear_pad(d)], v float32 [T, H*dv] (rows may be strided), g float32 [T, H] or [H] (the same for every token),
-    gate float32 [T, H*dv] logits (rows may be strided), norm float32 [dv] or None; S [H, dv, d] float32 at ``s_off`` of
-    the request's row of ``state``; out [T, H*dv] (rows may be strided)."""
-    T, G, DP = q.shape
-    assert q.dtype == k.dtype == v.dtype == g.dtype == gate.dtype == torch.float32 and k.shape == q.shape
-    assert v.shape == gate.shape == out.shape == (T, H * dv) and v.stride(1) == gate.stride(1) == out.stride(1) == 1
-    assert g.shape in ((T, H), (H,)) and (beta is None or (beta.shape == (T, H) and beta.dtype == torch.float32))
-    assert norm is None or (norm.dtype == torch.float32 and norm.numel() == dv)
-    assert state.dtype == torch.float32 and s_off + H * dv * d <= state.shape[1]
-    for n, t in (("q", q), ("k", k), ("g", g), ("state", state)):
-        _contig(t, n)
+    S <- S + k x^T;  o = S^T q;  out[t, head] = o / sqrt(mean(o^2) + eps) * norm * silu(gate) * out_scale (``gate_kind`` 1:
+    sigmoid(gate)).  q, k float32 [T, G, linear_pad(d)], v float32 [T, H*dv] (rows may be strided), g float32 [T, H] or [H]
+    (the same for every token), gate float32 [T, H*dv] logits (rows may be strided), norm float32 [dv], [H*dv] or None;
+    S [H, dv, d] float32 at ``s_off`` of the request's row of ``state``; out [T, H*dv] (rows may be strided).
+
+    ``exp_gates``: S <- g S + k v^T and n <- g n + k, o = S^T q / (max(|n . q|, low) + 1e-6) with the n of a head as column dv of
+    its S [dv + 1, d]; for portions g, low and the factor that k already carries come from ``linear_exp_gates``, single
+    tokens work them out in the same launch (g and low None, k plain).
+
+    Single tokens also take q and k as they stand in a wider product: [T, G*d] (rows may be strided), times ``q_scale`` and
+    ``k_scale``."""
+    T = q.shape[0]
     single = T == ctx.num_requests
-    o = None if single else torch.empty((T, H * dv), dtype=torch.float32, device=q.device)
-    coef = None if single or beta is None else torch.empty((T, H, 12), dtype=torch.float32, device=q.device)
+    raw = q.dim() == 2
+    if raw:
+        assert single and k.shape == q.shape and q.stride(1) == k.stride(1) == 1 and q.stride(0) == k.stride(0)
+        G, DP = q.shape[1] // d, linear_pad(d)
+        assert q.shape[1] == G * d
+    else:
+        _, G, DP = q.shape
+        assert k.shape == q.shape and q_scale == k_scale == 1.0
+        _contig(q, "q"); _contig(k, "k")
+    nrm = 1 if exp_gates is not None else 0
+    assert q.dtype == k.dtype == v.dtype == gate.dtype == torch.float32
+    assert v.shape == gate.shape == out.shape == (T, H * dv) and v.stride(1) == gate.stride(1) == out.stride(1) == 1
+    if g is None:
+        assert nrm and single
+    else:
+        assert g.dtype == torch.float32 and g.shape in ((T, H), (H,))
+        _contig(g, "g")
+    assert beta is None or (beta.shape == (T, H) and beta.dtype == torch.float32)
+    assert norm is None or (norm.dtype == torch.float32 and norm.is_contiguous() and norm.numel() in (dv, H * dv))
+    assert state.dtype == torch.float32 and s_off + H * (dv + nrm) * d <= state.shape[1]
+    _contig(state, "state")
+    e = exp_gates
+    if nrm:
+        assert beta is None and G == H and e.m_off + H <= state.shape[1]
+        assert single or (low is not None and low.shape == (T, H) and low.dtype == torch.float32 and low.is_contiguous())
+    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=q.device)
+    o = None if single else new(T, H * dv)
+    nq = new(T, H) if nrm and not single else None
+    coef = None if single or beta is None else new(T, H, 12)
     _check(library("linear_scan").qd_linear_scan(
-        _ptr(q), _ptr(k), _ptr(v), _LL(v.stride(0)), _ptr(g), _I(H if g.dim() == 2 else 0), _ptr(beta), _I(T),
+        _ptr(q), _ptr(k), _ptr(v), _LL(v.stride(0)), _ptr(g), _I(H if g is not None and g.dim() == 2 else 0), _ptr(beta), _I(T),
         _I(ctx.num_requests), _I(H), _I(G), _I(d), _I(dv), _I(DP), _ptr(state), _LL(state.stride(0)), _LL(s_off),
         _ptr(ctx.cu_tokens), _ptr(ctx.state_slots), _I(1 if write_state else 0), _ptr(o), _ptr(gate), _LL(gate.stride(0)),
         _ptr(norm), _F(eps), _F(out_scale), _ptr(out), _I(dtype_code(out.dtype)), _LL(out.stride(0)), _ptr(ctx.token_request),
-        _ptr(coef), _stream()), "linear_scan")
+        _ptr(coef), _I(dv if norm is not None and norm.numel() == H * dv else 0), _I(gate_kind), _I(nrm), _ptr(nq), _ptr(low),
+        _ptr(e.u if nrm else None), _LL(e.u.stride(0) if nrm else 0), _I(e.i_off if nrm else 0), _I(e.f_off if nrm else 0),
+        _ptr(e.i_bias if nrm else None), _ptr(e.f_bias if nrm else None), _F(e.cap if nrm else 1.0), _LL(e.m_off if nrm else 0),
+        _I(1 if raw else 0), _LL(q.stride(0) if raw else 0), _F(q_scale), _F(k_scale), _stream()), "linear_scan")
     if not single:
         _launch_count[0] += 1 if coef is None else 2
 
@@ -1524,7 +1603,7 @@ def group_add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], post=None, de
     """x += y, y = delta (+ ``delta_bias`` [D]; delta [T, D], or float32 partial sums [n, T, D] that are added up), or with
     ``post`` = (w, eps, groups) x += G(y; w, eps, groups); with ``weight`` also out[r] = G(x[s]; weight, eps, groups),
     s = rows[r] (or r).  G cuts a row into ``groups`` equal parts, divides each by its own sqrt(mean(part^2) + eps) and
-    multiplies the whole by the weight.  ``write_back`` False leaves x as it was (the norm still sees the sum)."""
+    multiplies the whole by the weight.  ``out`` without ``weight``: out[r] = x[s], rounded.  ``write_back`` False leaves x as it was (the norm still sees the sum)."""
     T, D = x.shape
     assert x.dtype == torch.float32
     _contig(x, "x")
@@ -1539,7 +1618,8 @@ def group_add_norm(x: torch.Tensor, delta: Optional[torch.Tensor], post=None, de
     f32 = lambda t: t is None or (t.dtype == torch.float32 and t.numel() == D and t.is_contiguous())
     assert f32(pw) and f32(delta_bias) and f32(weight)
     n_rows = T
-    if weight is not None:
+    assert weight is None or out is not None
+    if out is not None:
         n_rows = out.shape[0]
         assert out.shape == (n_rows, D) and (rows is None or (rows.dtype == torch.int32 and rows.numel() == n_rows))
         _contig(out, "out")

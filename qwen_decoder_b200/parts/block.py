@@ -352,6 +352,58 @@ class PrePostNormBlock(Block):
         stream.push(delta, post=self.norms[3].as_post(), bias=bias)
 
 
+@register_part("block", "post_norm")
+class PostNormBlock(Block):
+    """A norm on each branch's output and none before it: the branches read the residual sum itself (rounded to the
+    engine's dtype),
+
+        x += norm_out1(mixer(x));   x += norm_out2(feed_forward(x))      (a layer may have no feed-forward)
+
+    A branch's output waits on the stream with its norm; the launch that adds it also writes the rounded sum the next
+    branch reads."""
+    norm_roles = ("mixer_out", "feed_forward_out")
+
+    def __init__(self, mixer: Mixer, feed_forward, norms: Dict[str, Norm]):
+        need = self.norm_roles if feed_forward is not None else self.norm_roles[:1]
+        missing = [r for r in need if r not in norms]
+        if missing:
+            raise ValueError(f"post_norm block needs norms {need}, missing {missing}")
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.norms = [norms[r] for r in need]
+        for n in self.norms:
+            if not hasattr(n, "as_post"):
+                raise ValueError(f"post_norm block: {type(n).__name__} cannot norm a branch's output")
+
+    def parts(self):
+        return self.norms + [p for p in (self.mixer, self.feed_forward) if p is not None]
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [s for p in self.parts() for s in p.tensor_specs()]
+
+    def bind(self, source: TensorSource, dtype: torch.dtype, device: torch.device) -> None:
+        self.dtype = dtype
+        for p in self.parts():
+            p.bind(source, dtype, device)
+
+    def _sum(self, stream: ResidualStream) -> torch.Tensor:
+        """The residual sum with what was pending, in the engine's dtype."""
+        if self.dtype == torch.float32:
+            stream.flush()
+            return stream.x
+        stream.settle(post_ok=True)
+        if stream.delta_scale is not None:
+            stream.flush()
+        h = torch.empty(stream.x.shape, dtype=self.dtype, device=stream.x.device)
+        kernels.group_add_norm(stream.x, stream.delta, stream.delta_post, stream.delta_bias, out=h)
+        stream.clear()
+        return h
+
+    def forward(self, stream: ResidualStream, ctx, cache) -> None:
+        stream.push(self.mixer.forward(self._sum(stream), ctx, cache), post=self.norms[0].as_post())
+        if self.feed_forward is not None:
+            stream.push(self.feed_forward.forward(self._sum(stream), ctx), post=self.norms[1].as_post())
+
+
 @register_part("block", "loop_input")
 class LoopInput(Block):
     """What stands before every pass of a loop of layers: the residual sum takes the embedding output x0 in again

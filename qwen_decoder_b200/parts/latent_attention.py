@@ -152,7 +152,7 @@ class LatentAttention(Mixer):
         u = self.down.forward(x, out_dtype=torch.float32)                   # [T, qr (or q itself) | r + dr | H * dv]
         cq = torch.empty((T, qr), dtype=x.dtype, device=x.device)
         kernels.latent_prep(u, 0, qr, qw, r, dr, self.w_dq_norm, self.w_dkv_norm, self.eps, *rot, ctx.positions,
-                            cache.group.slot_map, cq, cache.kv, cache.write)
+                            cache.group.slot_map, cq, cache.kv, cache.write, pairing=pos.pairing_code if pos is not None else 0)
         q = self.up_q.forward(cq, out_dtype=torch.float32) if qr else u[:, :qw]
         attn = torch.empty((T, H * dv), dtype=x.dtype, device=x.device)
         # rows 0 .. Ta-1 take the absorbed form: all of them, or the single tokens of a step whose portions expand
@@ -184,7 +184,8 @@ class LatentAttention(Mixer):
             qn = _hi_lo(q.view(T, H, dn + dr)[:, :, :dn])                                   # [H, T, 2 dn]
             pre = torch.bmm(qn, self.w_uk_twice, out_dtype=torch.float32)                   # [H, T, r]
             matmul_backend.counters["library"] += 1
-        kernels.latent_absorb(q, self.w_uk, qcat, H, dn, dr, r, *rot, positions, pre=pre)
+        kernels.latent_absorb(q, self.w_uk, qcat, H, dn, dr, r, *rot, positions, pre=pre,
+                              pairing=pos.pairing_code if pos is not None else 0)
         o_lat = torch.empty((T, H, r), dtype=torch.float32, device=dev)
         window = self.window or 0
         groups = -(-H // 8)

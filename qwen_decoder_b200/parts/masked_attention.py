@@ -17,6 +17,7 @@ i // (H / G)), query/key size d and value size vd:
     s_ij = (q_i . k_j) * scale for the keys j <= i that the mask lets through:
         "causal" all of them;  "window" those with i - j < size;  "chunk" those with j // size == i // size
         (blocks counted from position 0 of the sequence, wherever a prompt was cut)
+    ``softcap`` c: s_ij <- c tanh(s_ij / c), before the mask
     o_i = softmax_j(s_ij) v_j;   ``sink_score`` s: exp(s) joins the softmax's denominator (a key of that score, no value)
     ``output_gate`` "head" (or True): head h's o times sigmoid(Wg h)_h (``g`` [H, D]);  "element": the concatenated heads
         times sigmoid(Wg h) element by element (``g`` [H*vd, D]);   out = Wo [o of all heads]
@@ -26,6 +27,11 @@ projected rows [q | k | v] before the convolution (float32).  q, k, v and the ga
 float32 sums; convolution, norms, rotation, scores and softmax weights are float32 in both engine dtypes
 (``csrc/qkv_prep.cu``, ``csrc/attention_sink.cu``).  A windowed mixer's pages are given back once the window has
 passed them.
+
+``shares_kv``: the layer has no keys and values of its own (no projections, convolutions or norms of them): its run reads
+another run's cache, keys as they were cached there, with its own queries, scale and mask.  ``cache_window``: how many
+positions the cache must keep readable where that is not the mask's size (a layer whose keys another layer reads
+through a wider window).
 
 ``inner`` computes everything up to the output projection into a tensor the caller gives (a column range of a wider
 one, say), times ``out_scale``: a mixer that runs beside another one shares one output product with it.
@@ -54,7 +60,8 @@ class MaskedAttention(Mixer):
                  scale: Optional[float] = None, eps: float = 1e-6, bias: bool = False, conv_taps: int = 0,
                  qk_norm: str = "none", norm_after_rotation: bool = True, position=None, mask: str = "causal",
                  mask_size: int = 0, output_gate=False, prefix: str = "mix.", weight_suffix: str = "",
-                 bias_suffix: str = ".b", output_projection: bool = True, sink_score: Optional[float] = None):
+                 bias_suffix: str = ".b", output_projection: bool = True, sink_score: Optional[float] = None,
+                 softcap: Optional[float] = None, shares_kv: bool = False, cache_window: Optional[int] = None):
         if num_heads % num_kv_heads:
             raise ValueError(f"masked_attention: kv heads ({num_kv_heads}) must divide heads ({num_heads})")
         if qk_norm not in kernels.QKV_NORMS or mask not in MASKS:
@@ -63,6 +70,14 @@ class MaskedAttention(Mixer):
             raise ValueError(f"masked_attention: output_gate must be one of {list(GATES)}, got {output_gate!r}")
         if mask != "causal" and mask_size < 1:
             raise ValueError(f"masked_attention: mask {mask!r} needs a size of at least 1")
+        if softcap is not None and not softcap > 0:
+            raise ValueError("masked_attention: softcap must be positive")
+        if shares_kv and conv_taps:
+            raise ValueError("masked_attention: a layer that reads another layer's keys has no convolution")
+        if cache_window is not None and (mask != "window" or cache_window < mask_size):
+            raise ValueError("masked_attention: cache_window goes with a window mask and is at least its size")
+        self.softcap, self.shares_kv = float(softcap or 0.0), bool(shares_kv)
+        self.cache_window = int(cache_window or mask_size or 0)
         self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
         self.head_dim, self.v_dim = head_dim, v_dim or head_dim
         self.scale = float(scale) if scale is not None else head_dim ** -0.5
@@ -72,8 +87,10 @@ class MaskedAttention(Mixer):
         self.output_gate, self.prefix, self.sfx = GATES[output_gate], prefix, weight_suffix
         self.sink_score, self.sinks = sink_score, None
         H, G, d, vd = num_heads, num_kv_heads, head_dim, self.v_dim
-        self.channels = H * d + G * d + G * vd
-        pieces = [(f"{prefix}q", H * d), (f"{prefix}k", G * d), (f"{prefix}v", G * vd)]
+        self.channels = H * d + (0 if shares_kv else G * d + G * vd)
+        pieces = [(f"{prefix}q", H * d)]
+        if not shares_kv:
+            pieces += [(f"{prefix}k", G * d), (f"{prefix}v", G * vd)]
         self.qkv = Linear(hidden_size, pieces, bias=self.has_bias, weight_suffix=weight_suffix, bias_suffix=bias_suffix)
         # the gate has no bias: a product of its own rows, stacked under q, k, v when bound
         self.gates = {None: 0, "head": H, "element": H * vd}[self.output_gate]
@@ -90,7 +107,7 @@ class MaskedAttention(Mixer):
         return (self.conv_taps - 1) * self.channels if self.conv_taps > 1 else 0
 
     def paged_need(self):
-        return PagedKV(self.num_kv_heads, self.head_dim, self.mask_size if self.mask == "window" else None,
+        return PagedKV(self.num_kv_heads, self.head_dim, self.cache_window if self.mask == "window" else None,
                        v_dim=self.v_dim)
 
     def cache_need(self):
@@ -109,8 +126,9 @@ class MaskedAttention(Mixer):
             specs += [TensorSpec(f"{p}{n}.conv", (c, self.conv_taps), init="uniform:-0.5:0.5")
                       for n, c in (("q", H * d), ("k", G * d), ("v", G * vd))]
         if self.qk_norm == "whole":
-            specs += [TensorSpec(f"{p}q.norm", (H * d,), init="around_one"),
-                      TensorSpec(f"{p}k.norm", (G * d,), init="around_one")]
+            specs.append(TensorSpec(f"{p}q.norm", (H * d,), init="around_one"))
+            if not self.shares_kv:
+                specs.append(TensorSpec(f"{p}k.norm", (G * d,), init="around_one"))
         return specs
 
     def bind(self, source: TensorSource, dtype: torch.dtype, device: torch.device) -> None:
@@ -131,7 +149,8 @@ class MaskedAttention(Mixer):
         if self.conv_taps:
             self.conv_w = torch.cat([f32(f"{p}{n}.conv") for n in ("q", "k", "v")], dim=0).contiguous()
         if self.qk_norm == "whole":
-            self.w_q_norm, self.w_k_norm = f32(f"{p}q.norm"), f32(f"{p}k.norm")
+            self.w_q_norm = f32(f"{p}q.norm")
+            self.w_k_norm = None if self.shares_kv else f32(f"{p}k.norm")
 
     def release_inputs(self) -> None:
         """``stacked`` is now a view of a larger matrix: let go of the copies it was stacked from."""
@@ -157,14 +176,17 @@ class MaskedAttention(Mixer):
         rope = (pos.rotary_dim, pos.pairing_code, pos.cos, pos.sin) if pos is not None else (0, 0, None, None)
         q = torch.empty((T, H * d), dtype=x.dtype, device=x.device)
         grp = paged.group
-        kernels.qkv_prep(u, H, G, d, vd, self.conv_w, state, state_off, ctx, paged.write, self.qk_norm, self.norm_after,
+        if self.shares_kv and paged.write:
+            raise ValueError("masked_attention: shares_kv needs a run that reads another run's cache")
+        kernels.qkv_prep(u, H, 0 if self.shares_kv else G, d, vd, self.conv_w, state, state_off, ctx, paged.write, self.qk_norm, self.norm_after,
                          self.w_q_norm, self.w_k_norm, self.eps, *rope, q, paged.kv, grp.slot_map, grp.page_size,
                          paged.write)
         gate = u[:, self.channels:self.channels + self.gates] if self.gates else None
         window = self.mask_size if self.mask == "window" else 0
         chunk = self.mask_size if self.mask == "chunk" else 0
         ps = grp.page_size
-        extra = dict(chunk=chunk, gate=gate, out_scale=out_scale, gate_elem=self.output_gate == "element")
+        extra = dict(chunk=chunk, gate=gate, out_scale=out_scale, gate_elem=self.output_gate == "element",
+                     cap=self.softcap)
         if _TENSOR_CORES and kernels.sink_mma_supported(x.dtype, H, G, d, vd):
             args = (H, G, d, vd, ps, self.scale, window, self.sinks)
             nd = T if ctx.all_decode else getattr(ctx, "num_decode", 0)

@@ -4,7 +4,8 @@ W1 = gate_proj, W3 = up_proj, W2 = down_proj).  Gate and up are one stacked prod
 
 ``activation`` = "clamped" (with ``limit`` L and ``alpha`` a; the reference has silu only) gates instead with
 g = min(x W1^T, L), u = clamp(x W3^T, -L, L), h = g * sigmoid(a g) * (u + 1); the stacked product then leaves
-float32 sums and one elementwise kernel makes h.
+float32 sums and one elementwise kernel makes h.  ``activation`` = "gelu_tanh" puts
+gelu(z) = 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) in silu's place, in every fused form.
 """
 from __future__ import annotations
 
@@ -20,7 +21,7 @@ from . import matmul_backend
 from .linear import Linear
 
 
-ACTIVATIONS = {"silu": kernels.ACT_SILU, "clamped": kernels.ACT_CLAMPED}
+ACTIVATIONS = {"silu": kernels.ACT_SILU, "clamped": kernels.ACT_CLAMPED, "gelu_tanh": kernels.ACT_GATED_GELU}
 
 
 @register_part("feed_forward", "swiglu")
@@ -80,28 +81,28 @@ class SwiGLU(FeedForward):
         return self.down.forward_partial(h, with_bias=False)
 
     def _products(self, x: torch.Tensor) -> torch.Tensor:
-        if self.activation != "silu":
+        act = ACTIVATIONS[self.activation]
+        if self.activation == "clamped":
             h = torch.empty((x.shape[0], self.intermediate_size), dtype=x.dtype, device=x.device)
-            kernels.gated_act(self.gate_up.forward(x, out_dtype=torch.float32), h, ACTIVATIONS[self.activation],
-                              self.limit, self.alpha)
+            kernels.gated_act(self.gate_up.forward(x, out_dtype=torch.float32), h, act, self.limit, self.alpha)
             return self._down(h)
         if matmul_backend.mode == "auto" and kernels.ffn_stream_supported(x, self.gate_up.weight, self.down.weight):
             matmul_backend.counters["own"] += 1
             if self._barrier is None:       # this layer's own synchronisation words (zero once; each launch leaves them zero)
                 self._barrier = torch.zeros(kernels.FFN_SYNC_WORDS, dtype=torch.int32, device=x.device)
             return kernels.ffn_stream(x, self.gate_up.weight, self.down.weight, self._barrier,
-                                      bias=self.gate_up.bias)   # one launch
+                                      bias=self.gate_up.bias, act=act)   # one launch
         h = torch.empty((x.shape[0], self.intermediate_size), dtype=x.dtype, device=x.device)
         if matmul_backend.use_skinny(x, self.gate_up.weight):
             shares = kernels.swiglu_shares(x.shape[0], self.hidden_size, 2 * self.intermediate_size)
             if shares and self.intermediate_size % 4 == 0:
                 # where the streamer keeps the tokens resident only for a share of K: partial sums, then SwiGLU
-                kernels.swiglu_partial(kernels.gemm_skinny_partial(x, self.gate_up.weight, shares), h, self.gate_up.bias)
+                kernels.swiglu_partial(kernels.gemm_skinny_partial(x, self.gate_up.weight, shares), h, self.gate_up.bias, act)
             else:
-                kernels.gemm_skinny_swiglu(x, self.gate_up.weight, h, self.gate_up.bias)       # gate, up and SwiGLU in one kernel
+                kernels.gemm_skinny_swiglu(x, self.gate_up.weight, h, self.gate_up.bias, act)       # gate, up and the activation in one kernel
             matmul_backend.counters["own"] += 1
         else:
-            kernels.swiglu(self.gate_up.forward(x), h)
+            kernels.swiglu(self.gate_up.forward(x), h, act)
         return self._down(h)
 
 

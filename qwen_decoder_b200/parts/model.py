@@ -73,6 +73,7 @@ class DecoderModel:
         else:           # a model that names its output matrix without the suffix
             self.lm_head = Linear(spec.hidden_size, [(head, spec.vocab_size)], bias=False, weight_suffix="")
         self.embedding_scale = float(spec.embedding_scale)
+        self.logit_softcap = spec.logit_softcap
         self.embedding: Optional[torch.Tensor] = None
         self.native_prompt = None    # parts.native_prompt.NativePrompt once bound, if the parts allow it
         self.dtype: Optional[torch.dtype] = None
@@ -171,7 +172,7 @@ class DecoderModel:
             h = self.native_prompt.forward(ctx, x)
             if h is None:
                 return torch.empty((0, self.vocab_size), dtype=torch.float32, device=self.device)
-            return self.lm_head.forward(h, out_dtype=torch.float32)
+            return self._logits(h)
         stream = ResidualStream(x)
         if self.keeps_origin:
             stream.origin = x.clone()
@@ -184,7 +185,13 @@ class DecoderModel:
         if ctx.num_wanted == 0:
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=self.device)
         h = self.final_norm.forward(stream, self.dtype, rows=ctx.logit_rows)
-        return self.lm_head.forward(h, out_dtype=torch.float32)
+        return self._logits(h)
+
+    def _logits(self, h: torch.Tensor) -> torch.Tensor:
+        logits = self.lm_head.forward(h, out_dtype=torch.float32)
+        if self.logit_softcap is not None:
+            kernels.soft_cap(logits, self.logit_softcap)
+        return logits
 
 
 def build_model(spec: ModelSpec) -> DecoderModel:

@@ -10,6 +10,7 @@ by the plain scores, not renormalised (no router bias); the last ``identity`` ou
 experts without tensors, expert(h) = h; ``activation`` = "clamped" with ``limit`` and ``alpha`` is the gate of
 ``parts.mlp`` (the shared expert has its own ``shared_limit``); ``shared_gate`` = False adds the shared expert in full.
 ``routing`` = "top_sigmoid" chooses the ``top`` largest logits and weighs each by its own sigmoid, not renormalised;
+"top_sigmoid_norm" divides those by their sum (+ 1e-20); all weights are multiplied by ``routing_scale``;
 ``router_bias`` = False leaves the router without a bias; ``weigh`` = "input" lets a pair's weight multiply the
 expert's input instead of its output, out = sum_k expert_k(weight_k h) (the gate is not linear, so this differs):
 since W (w h) = w (W h), the grouped product multiplies the pair's two sums by w before the gate.
@@ -32,7 +33,7 @@ from . import matmul_backend
 from .mlp import ACTIVATIONS, SwiGLU
 
 ROUTINGS = {"top_softmax": kernels.MOE_ROUTE_TOP_SOFTMAX, "softmax_all": kernels.MOE_ROUTE_SOFTMAX_ALL,
-            "top_sigmoid": kernels.MOE_ROUTE_TOP_SIGMOID}
+            "top_sigmoid": kernels.MOE_ROUTE_TOP_SIGMOID, "top_sigmoid_norm": kernels.MOE_ROUTE_TOP_SIGMOID_NORM}
 
 
 @register_part("feed_forward", "moe")
@@ -41,7 +42,7 @@ class RoutedExperts(FeedForward):
                  prefix: str = "mlp.", weight_suffix: str = ".weight", names=("gate", "up", "down"),
                  routing: str = "top_softmax", identity: int = 0, activation: str = "silu", limit: float = 0.0,
                  alpha: float = 1.0, shared_limit: float = 0.0, shared_gate: bool = True, router_bias: bool = True,
-                 weigh: str = "output"):
+                 weigh: str = "output", routing_scale: float = 1.0):
         outputs = num_experts + identity
         if not (1 <= top <= outputs) or top > kernels.MOE_MAX_TOP:
             raise ValueError(f"moe: top ({top}) must be between 1 and the router's outputs ({outputs}), at most {kernels.MOE_MAX_TOP}")
@@ -51,6 +52,7 @@ class RoutedExperts(FeedForward):
         if weigh not in ("output", "input") or (weigh == "input" and identity):
             raise ValueError("moe: weigh must be 'output' or 'input' (and 'input' goes without identity experts)")
         self.identity, self.outputs = identity, outputs
+        self.routing_scale = float(routing_scale)
         self.router_bias, self.weigh = bool(router_bias) and routing != "softmax_all", weigh
         self.routing, self.activation, self.limit, self.alpha = routing, activation, float(limit), float(alpha)
         self.prefix, self.sfx, self.names = prefix, weight_suffix, tuple(names)
@@ -112,10 +114,10 @@ class RoutedExperts(FeedForward):
             # whichever kernel takes a product of this many tokens; then the choice
             logits = torch.empty((T, O), dtype=torch.float32, device=dev)
             matmul_backend.linear(x, self.w_router, None, logits)
-            kernels.moe_choose(logits, top, idx, wt, ROUTINGS[self.routing], self.correction)
+            kernels.moe_choose(logits, top, idx, wt, ROUTINGS[self.routing], self.correction, self.routing_scale)
         else:
             kernels.moe_route(x, self.w_router, self.b_router, self.w_sg, top, idx, wt, sgate, ROUTINGS[self.routing],
-                              self.correction)
+                              self.correction, self.routing_scale)
         tile_rows = kernels.moe_tile_rows(n, E, D, F, x.dtype)   # rows of one expert a CTA takes
         max_tiles = n // tile_rows + E              # sum over experts of ceil(count / tile_rows) is at most this
         place = torch.empty((n,), dtype=torch.int32, device=dev)
