@@ -423,6 +423,44 @@ def gopevik_configs(size, layers=None):
     return gopevik, fogurax
 
 
+# ---- Furesun beside Fogurax at equal layer sizes ----------------------------------------------------------------------
+# Eight layers, twice: a matrix memory (width / 64 heads of 64) + dense feed-forward, windowed attention + routed experts, the same
+# over the keys and values of the layer before it, latent attention in a window + routed experts.  Heads of 128 with values of 128,
+# windows of 1,024 positions, latent rows of 512 + 64.  The other model: Fogurax (windowed and block-masked attention on the same
+# kernels, a recurrent mixer with a matrix state per head, the same feed-forwards) with the same width, depth, heads, windows,
+# recurrent heads, feed-forward sizes and vocabulary.  The latent attention's like is Zunuvik's (--micro hybrid).
+FURESUN_SIZES = {
+    "S": dict(FOGURAX_SIZES["S"], latent=dict(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512)),
+    "M": dict(FOGURAX_SIZES["M"], latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512)),
+}
+
+
+def furesun_configs(size, layers=None):
+    from qwen_decoder_b200.config import config_from_dict
+    z = FURESUN_SIZES[size]
+    (H, G), d, n, m = z["heads"], z["dim"], z["width"] // 64, z["moe"]
+    count = max(1, layers or 8)     # fewer layers of the same sizes: a capture under a profiler holds fewer weights
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": m["ff"]}, "router": {"experts": m["experts"], "top": m["top"]}, "shared": {"ff": m["shared"]}}
+    scaled = dict(moe, router=dict(moe["router"], scale=1.5))
+    base = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5}
+    attn = dict(base, mask={"size": z["span"]}, softcap=30.0, rot={"base": 200000.0, "dims": d // 2})
+    latent = dict(z["latent"], mask={"size": z["span"]}, scale=(z["latent"]["dim"] + z["latent"]["rot_dim"]) ** -0.5,
+                  rot={"base": 200000.0, "dims": z["latent"]["rot_dim"], "scaling": {"factor": 4.0, "original": 4096, "fast": 16.0, "slow": 2.0}})
+    layer = lambda kind, mixer, mlp: {"type": kind, "mixer": mixer, "mlp": mlp}
+    four = lambda at: [layer("mlstm", {"heads": n, "dim": 64, "vdim": 64, "gate_cap": 15.0}, dense), layer("attention", attn, scaled),
+                       layer("attention", dict(attn, kv_from=at + 1), scaled), layer("latent_attention", latent, scaled)]
+    furesun = config_from_dict({"architecture": "Furesun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+                                "logit_softcap": 30.0, "layers": (four(0) + four(4))[:count]})
+    mixed = {"type": "parallel", "mixer": {
+        "left": dict(base, mask={"size": z["span"]}, rot={"base": 10000.0, "dims": d}), "right": {"heads": n, "dim": 64, "rank": z["rank"]},
+        "left_scale": 0.8, "right_scale": 1.25}}
+    block = {"type": "attention_2", "mixer": dict(base, mask={"size": z["span"]}, rot={"base": 200000.0, "dims": d // 2})}
+    fogurax = config_from_dict({"architecture": "Fogurax", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+                                "layers": ([dict(mixed, mlp=dense), dict(block, mlp=moe), dict(block, mlp=moe), dict(block, mlp=moe)] * 2)[:count]})
+    return furesun, fogurax
+
+
 def hybrid_bench(args, label="hybrid", configs=None, other="dense"):
     """``--micro hybrid`` (and ``--micro veterax``, which passes its own pair of models): decode steps (batch 1, 8, 64 at ``--context``) and a prompt of ``--prefill-tokens`` tokens, for the
     hybrid design and for the dense decoder at equal sizes; one JSON line.  ``--only hybrid|dense`` and ``--phase`` narrow it
@@ -576,6 +614,8 @@ def micro(args):
         return hybrid_bench(args, "fogurax", lambda size: fogurax_configs(size, args.veterax_layers), other="veterax")
     if args.micro == "gopevik":
         return hybrid_bench(args, "gopevik", lambda size: gopevik_configs(size, args.veterax_layers), other="fogurax")
+    if args.micro == "furesun":
+        return hybrid_bench(args, "furesun", lambda size: furesun_configs(size, args.veterax_layers), other="fogurax")
     if args.micro == "latent_attend":
         return latent_attend_micro(args)
     """One kernel alone: W-streaming contraction, decode attention or prefill attention at the 3B sizes."""
@@ -827,7 +867,7 @@ def main():
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--timeline", action="store_true",
                     help="with --micro prefill_attention: print the kernel's own time stamps of one CTA (microseconds) to stderr")
-    ap.add_argument("--micro", default=None, choices=["gemm", "decode_attention", "decode_attention_rope", "prefill_attention", "serve", "mixed_step", "hybrid", "latent_attend", "veterax", "solopel", "fogurax", "gopevik"],
+    ap.add_argument("--micro", default=None, choices=["gemm", "decode_attention", "decode_attention_rope", "prefill_attention", "serve", "mixed_step", "hybrid", "latent_attend", "veterax", "solopel", "fogurax", "gopevik", "furesun"],
                     help="time one kernel alone at the 3B shape (for profiles/), or with 'serve' a whole run of "
                          "--batch requests (--context prompt tokens, --steps new tokens each) through the entry "
                          "point; print one JSON line and exit")
@@ -841,7 +881,7 @@ def main():
     ap.add_argument("--micro-splits", type=int, default=1, help="gemm with --micro-graph: shares of K (partial sums)")
     ap.add_argument("--hybrid-size", default="S", choices=["S", "M"], help="hybrid, veterax, solopel: which layer sizes")
     ap.add_argument("--only", default=None, choices=["hybrid", "dense", "other"], help="hybrid, veterax, solopel: one of the two models (hybrid = the first; dense, other = the second)")
-    ap.add_argument("--veterax-layers", type=int, default=None, help="veterax, solopel, fogurax, gopevik: fewer layers than the size has")
+    ap.add_argument("--veterax-layers", type=int, default=None, help="veterax, solopel, fogurax, gopevik, furesun: fewer layers than the size has")
     ap.add_argument("--phase", default="all", choices=["all", "decode", "prefill"], help="hybrid: decode steps, the prompt, or both")
     ap.add_argument("--history", type=int, default=2048, help="mixed_step: cached tokens before the prompt portion")
     ap.add_argument("--stamps", action="store_true",

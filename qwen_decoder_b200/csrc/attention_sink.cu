@@ -291,8 +291,8 @@ extern "C" int qd_sink_attention_generic(const void* q, long long q_stride, void
 // pairs, 64 / group tokens of them, so every row reads the same keys and values, which arrive in tiles of 64 keys by
 // 16-byte cp.async (two stages) through the block table, key by key: any page size.  Scores stay float32; a softmax
 // weight enters P V as TWO bfloat16 numbers (p = hi + lo, two products into one float32 sum), so weights keep 16 bits
-// of mantissa.  Head sizes are padded with zero columns in shared memory up to the template's D (keys: 64, 128) and DV
-// (values: 64, 96, 128): any multiple of 8 up to 128 runs.  With ``splits`` > 1 the key tiles of a CTA's range are shared among
+// of mantissa.  Head sizes are padded with zero columns in shared memory up to the template's D (keys: 64, 128, 192) and DV
+// (values: 64, 96, 128): any multiple of 8 up to 192 (keys) and 128 (values) runs.  With ``splits`` > 1 the key tiles of a CTA's range are shared among
 // gridDim.z CTAs that leave (o, m, l) per row in scratch memory; the CTA that finishes last for a tile (a ticket per
 // tile) adds them up with the sink (``sink_combine_kernel`` does, where there are no tickets); with one split the kernel
 // finishes the rows itself.
@@ -650,7 +650,7 @@ extern "C" int qd_sink_attention_mma(const void* q, void* out, const void* kv, c
                                      unsigned* tickets, int chunk, const float* gate, long long gate_ld,
                                      int gate_elem, float out_scale, long long out_stride, float cap, cudaStream_t stream) {
   if (n_tokens <= 0 || n_requests <= 0) return 0;
-  if (G <= 0 || H % G || H / G > TS_ROWS || d <= 0 || vd <= 0 || d > 128 || vd > 128 || d % 8 || vd % 8 ||
+  if (G <= 0 || H % G || H / G > TS_ROWS || d <= 0 || vd <= 0 || d > 192 || vd > 128 || d % 8 || vd % 8 ||
       page_size <= 0 || splits < 1 || splits > 64 || G > 65535 || (splits > 1 && (!part_o || !part_ml)) ||
       out_stride < (long long)H * vd || (out_stride & 1))
     return QD_ERR_UNSUPPORTED;
@@ -676,6 +676,7 @@ extern "C" int qd_sink_attention_mma(const void* q, void* out, const void* kv, c
   } while (0)
   if (d <= 64 && vd <= 64) TS_GO(64, 64);
   else if (d <= 64) TS_GO(64, 128);
+  else if (d > 128) TS_GO(192, 128);
   else if (vd <= 64) TS_GO(128, 64);
   else if (vd <= 96) TS_GO(128, 96);
   else TS_GO(128, 128);

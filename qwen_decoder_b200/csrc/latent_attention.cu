@@ -132,9 +132,9 @@ latent_absorb_kernel(const float* __restrict__ q, long long ldq, const TW* __res
   }
 }
 
-// The same with 16-byte loads of Wuk, for latent sizes whose pieces divide the CTA evenly (r / V a divisor of 256):
+// The same with 16-byte loads of Wuk, for latent sizes whose pieces divide the CTA evenly (a share's r / V a divisor of 256):
 // thread (jg, dg) owns V consecutive latent columns and every (256 * V / r)-th unrotated dimension; the groups'
-// partial sums meet in shared memory.  grid (token tiles, heads).
+// partial sums meet in shared memory.  grid (token tiles, heads, shares of the r columns).
 template <typename TW>
 __global__ void __launch_bounds__(256)
 latent_absorb_vec_kernel(const float* __restrict__ q, long long ldq, const TW* __restrict__ wuk,
@@ -146,25 +146,25 @@ latent_absorb_vec_kernel(const float* __restrict__ q, long long ldq, const TW* _
   constexpr int V = Vec16<TW>::N;
   extern __shared__ float sm[];
   float* qs = sm;                              // [LA_TT][dn]
-  float* red = sm + LA_TT * dn;                // [LA_TT][r]
+  float* red = sm + LA_TT * dn;                // [LA_TT][rs]
   const int h = blockIdx.y, t0 = blockIdx.x * LA_TT;
   const int nt = min(LA_TT, T - t0);
-  const int W = r + dr;
+  const int W = r + dr, rs = r / gridDim.z, j0 = blockIdx.z * rs;      // this CTA's columns
   const size_t qw = (size_t)ldq;              // q's rows are ldq floats apart (a column range of a wider buffer is fine)
   for (int i = threadIdx.x; i < LA_TT * dn; i += blockDim.x) {
     int tt = i / dn, d = i - tt * dn;
     qs[i] = tt < nt ? q[(size_t)(t0 + tt) * qw + (size_t)h * (dn + dr) + d] : 0.f;
   }
-  for (int i = threadIdx.x; i < LA_TT * r; i += blockDim.x) red[i] = 0.f;
+  for (int i = threadIdx.x; i < LA_TT * rs; i += blockDim.x) red[i] = 0.f;
   __syncthreads();
-  const int JG = r / V, DG = 256 / JG;
+  const int JG = rs / V, DG = 256 / JG;
   const int jg = threadIdx.x % JG, dg = threadIdx.x / JG;
   float acc[LA_TT][V];
 #pragma unroll
   for (int tt = 0; tt < LA_TT; tt++)
 #pragma unroll
     for (int v = 0; v < V; v++) acc[tt][v] = 0.f;
-  const TW* wbase = wuk + (size_t)h * dn * r + jg * V;
+  const TW* wbase = wuk + (size_t)h * dn * r + j0 + jg * V;
 #pragma unroll 4
   for (int d = dg; d < dn; d += DG) {
     float w[V];
@@ -181,14 +181,15 @@ latent_absorb_vec_kernel(const float* __restrict__ q, long long ldq, const TW* _
 #pragma unroll
       for (int tt = 0; tt < LA_TT; tt++)
 #pragma unroll
-        for (int v = 0; v < V; v++) red[tt * r + jg * V + v] += acc[tt][v];
+        for (int v = 0; v < V; v++) red[tt * rs + jg * V + v] += acc[tt][v];
     }
     __syncthreads();
   }
-  for (int i = threadIdx.x; i < nt * r; i += blockDim.x) {
-    int tt = i / r, j = i - tt * r;
-    qcat[((size_t)(t0 + tt) * H + h) * W + j] = red[i];
+  for (int i = threadIdx.x; i < nt * rs; i += blockDim.x) {
+    int tt = i / rs, j = i - tt * rs;
+    qcat[((size_t)(t0 + tt) * H + h) * W + j0 + j] = red[i];
   }
+  if (blockIdx.z != 0) return;
   const int half = rot_dims >> 1;
   for (int i = threadIdx.x; i < nt * dr; i += blockDim.x) {
     int tt = i / dr, e = i - tt * dr;
@@ -535,7 +536,7 @@ latent_expand_kernel(const float* __restrict__ o_lat, const TW* __restrict__ wuv
                      const float* __restrict__ pre) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float os[];                // [LA_TT][r]
+  extern __shared__ __align__(16) float os[];  // [LA_TT][r]
   const int h = blockIdx.y, t0 = blockIdx.x * LA_TT;
   const int nt = min(LA_TT, T - t0);
   const int i_hi = min(dv, (int)(blockIdx.z + 1) * 32);
@@ -568,7 +569,10 @@ latent_expand_kernel(const float* __restrict__ o_lat, const TW* __restrict__ wuv
 #pragma unroll
         for (int tt = 0; tt < LA_TT; tt++)
 #pragma unroll
-          for (int v = 0; v < V; v++) acc[tt] = fmaf(w[v], os[tt * r + j + v], acc[tt]);
+          for (int v = 0; v < V; v += 4) {
+            const float4 o = *reinterpret_cast<const float4*>(os + tt * r + j + v);
+            acc[tt] = fmaf(w[v], o.x, fmaf(w[v + 1], o.y, fmaf(w[v + 2], o.z, fmaf(w[v + 3], o.w, acc[tt]))));
+          }
       }
     } else {
       for (int j = lane; j < r; j += 32) {
@@ -635,7 +639,12 @@ extern "C" int qd_latent_absorb(const float* q, long long ldq, const void* wuk, 
     const size_t vsm = (size_t)LA_TT * (dn + r) * sizeof(float);
     if (!pre && (w_dtype == QD_F32 || w_dtype == QD_BF16) && r % V == 0 && r / V <= 256 && 256 % (r / V) == 0 &&
         !((uintptr_t)wuk & 15) && vsm <= 48 * 1024) {
-      dim3 vgrid((T + LA_TT - 1) / LA_TT, H);
+      // few tokens: a head's columns are shared among CTAs while the grid leaves multiprocessors idle
+      int shares = 1;
+      while (shares < 4 && (long long)((T + LA_TT - 1) / LA_TT) * H * shares < 128 && r % (2 * shares * V) == 0 &&
+             r / V / (2 * shares) >= 8)
+        shares *= 2;
+      dim3 vgrid((T + LA_TT - 1) / LA_TT, H, shares);
       if (w_dtype == QD_F32)
         qd_launch(latent_absorb_vec_kernel<float>, vgrid, dim3(256), vsm, stream, q, ldq, (const float*)wuk, qcat, T, H, dn, dr,
                   r, cos_t, sin_t, rot_dims, positions, pairing);
@@ -726,58 +735,86 @@ extern "C" int qd_latent_expand(const float* o_lat, const void* wuv, int w_dtype
 // For prompt portions the keys and values of all heads are expanded from the cached rows by one product, and an
 // ordinary attention kernel runs over them.  ``latent_gather`` lays the first r elements of every cached row of the
 // requests' contexts out densely, request by request with Lmax rows each (rows past a request's context are zero):
-//   out[(q * Lmax + j), :] = cache row j of request q,  j < start_pos[q] + tokens of q in this step
+//   out[(q * Lmax + j), :] = cache row lo_q + j of request q,  lo_q + j < start_pos[q] + tokens of q in this step
+// with lo_q = 0, or with a window the first row that the portion's first token still sees.
 // grid (Lmax, requests), 128 threads.
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_gather_kernel(const T* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
                      const int* __restrict__ cu_tokens, const int* __restrict__ start_pos, int page_size, int W, int r,
-                     T* __restrict__ out, int Lmax) {
+                     T* __restrict__ out, int Lmax, int window) {
   pdl_launch_dependents();
   pdl_wait();
   const int j = blockIdx.x, q = blockIdx.y;
-  const int len = start_pos[q] + cu_tokens[q + 1] - cu_tokens[q];
+  const int lo = window > 0 ? max(start_pos[q] - window + 1, 0) : 0;
+  const int len = start_pos[q] + cu_tokens[q + 1] - cu_tokens[q] - lo, key = lo + j;
   T* o = out + ((size_t)q * Lmax + j) * r;
   if (j >= len) {
     for (int i = threadIdx.x; i < r; i += blockDim.x) o[i] = from_float<T>(0.f);
     return;
   }
-  const int page = block_table[(size_t)q * max_blocks + j / page_size];
-  const T* src = cache + ((size_t)page * page_size + j % page_size) * W;
+  const int page = block_table[(size_t)q * max_blocks + key / page_size];
+  const T* src = cache + ((size_t)page * page_size + key % page_size) * W;
   for (int i = threadIdx.x; i < r; i += blockDim.x) o[i] = src[i];
 }
 
 extern "C" int qd_latent_gather(const void* cache, int dtype, const int* block_table, int max_blocks,
                                 const int* cu_tokens, const int* start_pos, int n_requests, int page_size, int W, int r,
-                                void* out, int Lmax, cudaStream_t stream) {
+                                void* out, int Lmax, int window, cudaStream_t stream) {
   if (n_requests <= 0 || Lmax <= 0) return 0;
   if (n_requests > 65535 || r <= 0 || r > W || page_size <= 0) return QD_ERR_UNSUPPORTED;
   dim3 grid(Lmax, n_requests);
   if (dtype == QD_BF16)
     qd_launch(latent_gather_kernel<bf16>, grid, dim3(128), 0, stream, (const bf16*)cache, block_table, max_blocks,
-              cu_tokens, start_pos, page_size, W, r, (bf16*)out, Lmax);
+              cu_tokens, start_pos, page_size, W, r, (bf16*)out, Lmax, window);
   else if (dtype == QD_F32)
     qd_launch(latent_gather_kernel<float>, grid, dim3(128), 0, stream, (const float*)cache, block_table, max_blocks,
-              cu_tokens, start_pos, page_size, W, r, (float*)out, Lmax);
+              cu_tokens, start_pos, page_size, W, r, (float*)out, Lmax, window);
   else
     return QD_ERR_UNSUPPORTED;
   return qd_last_error();
 }
 
-// out[t, 0..N) = in[t, 0..N) rounded to bfloat16 (in float32, rows ldin apart; out dense).
+// The queries of the expanded form: out[t, h, :] = [q's unrotated part | its rotated part turned], rounded to bfloat16
+// (q float32, rows ldq apart; out dense).  grid (ceil(H (dn + dr) / 1024), tokens): four neighbouring elements a thread;
+// ``vec``: they lie in one part of one head and on a 16-byte boundary.
 __global__ void __launch_bounds__(256)
-round_rows_kernel(const float* __restrict__ in, long long ldin, bf16* __restrict__ out, int N, size_t n) {
+latent_queries_kernel(const float* __restrict__ q, long long ldq, bf16* __restrict__ out, int H, int dn, int dr,
+                      const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims, int pairing,
+                      const int* __restrict__ positions, int vec) {
   pdl_launch_dependents();
   pdl_wait();
-  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= n) return;
-  const size_t t = i / N;
-  out[i] = __float2bfloat16_rn(in[t * ldin + (i - t * N)]);
+  const int c0 = (blockIdx.x * 256 + threadIdx.x) * 4, d = dn + dr, N = H * d, t = blockIdx.y;
+  if (c0 >= N) return;
+  const float* row = q + (size_t)t * ldq;
+  bf16* o = out + (size_t)t * N;
+  const int half = rot_dims >> 1;
+  const size_t at = (size_t)positions[t] * half;
+  auto one = [&](int c) {
+    const int e = c % d;
+    return e < dn ? row[c] : la_turn(row + c - e + dn, e - dn, half, pairing, cos_t + at, sin_t + at);
+  };
+  if (!vec) {
+    for (int c = c0; c < min(c0 + 4, N); c++) o[c] = __float2bfloat16_rn(one(c));
+    return;
+  }
+  float4 v;
+  if (c0 % d < dn) v = *reinterpret_cast<const float4*>(row + c0);
+  else v = make_float4(one(c0), one(c0 + 1), one(c0 + 2), one(c0 + 3));
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 raw;
+  raw.x = *reinterpret_cast<const unsigned*>(&lo);
+  raw.y = *reinterpret_cast<const unsigned*>(&hi);
+  *reinterpret_cast<uint2*>(o + c0) = raw;
 }
 
-extern "C" int qd_round_rows(const float* in, long long ldin, void* out, int T, int N, cudaStream_t stream) {
-  if (T <= 0 || N <= 0) return 0;
-  const size_t n = (size_t)T * N;
-  qd_launch(round_rows_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, in, ldin, (bf16*)out, N, n);
+extern "C" int qd_latent_queries(const float* q, long long ldq, void* out, int T, int H, int dn, int dr, const float* cos_t,
+                                 const float* sin_t, int rot_dims, int pairing, const int* positions, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || dn <= 0 || dr < 0 || rot_dims < 0 || rot_dims > dr || rot_dims % 2) return QD_ERR_UNSUPPORTED;
+  if (T > 65535) return QD_ERR_UNSUPPORTED;
+  const int vec = dn % 4 == 0 && dr % 4 == 0 && ldq % 4 == 0 && !((uintptr_t)q & 15) && !((uintptr_t)out & 7);
+  qd_launch(latent_queries_kernel, dim3((H * (dn + dr) + 1023) / 1024, T), dim3(256), 0, stream, q, ldq, (bf16*)out, H, dn, dr,
+            cos_t, sin_t, rot_dims, pairing, positions, vec);
   return qd_last_error();
 }

@@ -217,72 +217,64 @@ struct ExpGates {
   long long m_off;                                            // head h's maximum is at m_off + h of a state row
   int on;
 };
-__device__ __forceinline__ void exp_gate_logs(const ExpGates& a, int t, int h, float& i, float& f) {
-  const float* row = a.u + (size_t)t * a.ld;
-  i = a.cap * tanhf((row[a.i_off + h] + a.ib[h]) / a.cap);
-  const float z = a.cap * tanhf((row[a.f_off + h] + a.fb[h]) / a.cap);
+__device__ __forceinline__ void exp_gate_logs(const ExpGates& a, float ui, float uf, int h, float& i, float& f) {
+  i = a.cap * tanhf((ui + a.ib[h]) / a.cap);
+  const float z = a.cap * tanhf((uf + a.fb[h]) / a.cap);
   f = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
 }
 
-// grid (H, requests), one warp: the maxima of a portion by a scan over (sum of f, maximum): what a run of tokens does to m is
-// m -> max(F + m, M), and runs compose.  A lane takes LG_RUN neighbouring tokens.  Every factor is made from the maxima as
-// they are handed on, so what rounds in the scan cancels between a token and the next.
-#define LG_RUN 8
-__global__ void __launch_bounds__(32)
+// grid (H, requests): the maxima of a portion by a scan over (sum of f, maximum): what a run of tokens does to m is
+// m -> max(F + m, M), and runs compose.  A thread takes one token of LG_TOKENS; warps scan their 32, then one another's.
+// Every factor is made from the maxima as they are handed on, so what rounds in the scan cancels between a token and the next.
+#define LG_TOKENS 256
+__global__ void __launch_bounds__(LG_TOKENS)
 linear_exp_gates_kernel(ExpGates a, int H, float* __restrict__ state, long long state_stride,
                         const int* __restrict__ cu_tokens, const int* __restrict__ slots, int write_state,
                         float* __restrict__ g, float* __restrict__ in, float* __restrict__ low) {
   pdl_launch_dependents();
   pdl_wait();
-  const int h = blockIdx.x, req = blockIdx.y, lane = threadIdx.x;
+  __shared__ float wF[LG_TOKENS / 32], wM[LG_TOKENS / 32], ms[LG_TOKENS + 1];
+  const int h = blockIdx.x, req = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int t0 = cu_tokens[req], t1 = cu_tokens[req + 1];
   if (t0 >= t1) return;
   float* kept = state + (size_t)slots[req] * state_stride + a.m_off + h;
   float m0 = *kept;
-  for (int tb = t0; tb < t1; tb += 32 * LG_RUN) {
-    float iv[LG_RUN], fv[LG_RUN], F = 0.f, M = -INFINITY;
-#pragma unroll
-    for (int j = 0; j < LG_RUN; j++) {
-      const int t = tb + lane * LG_RUN + j;
-      iv[j] = -INFINITY;                              // past the end: m stays as it is
-      fv[j] = 0.f;
-      if (t < t1) exp_gate_logs(a, t, h, iv[j], fv[j]);
-      F += fv[j];
-      M = fmaxf(M + fv[j], iv[j]);
-    }
-    float Fs = F, Ms = M;                             // of all lanes up to this one
+  float ui = 0.f, uf = 0.f;                           // the logits of the turn ahead are under way during this one
+  auto fetch = [&](int t) {
+    if (t < t1) { ui = a.u[(size_t)t * a.ld + a.i_off + h]; uf = a.u[(size_t)t * a.ld + a.f_off + h]; }
+  };
+  fetch(t0 + tid);
+  for (int tb = t0; tb < t1; tb += LG_TOKENS) {
+    const int t = tb + tid;
+    float i = -INFINITY, f = 0.f;                     // past the end: m stays as it is
+    if (t < t1) exp_gate_logs(a, ui, uf, h, i, f);
+    fetch(t + LG_TOKENS);
+    float F = f, M = i;                               // of the warp's tokens up to this one
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float Fp = __shfl_up_sync(0xffffffffu, Fs, o), Mp = __shfl_up_sync(0xffffffffu, Ms, o);
+      const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
       if (lane >= o) {
-        Ms = fmaxf(Mp + Fs, Ms);
-        Fs += Fp;
+        M = fmaxf(Mp + F, M);
+        F += Fp;
       }
     }
-    float Fb = __shfl_up_sync(0xffffffffu, Fs, 1), Mb = __shfl_up_sync(0xffffffffu, Ms, 1);
-    float m = lane ? fmaxf(Fb + m0, Mb) : m0;         // before this lane's run
-    float mv[LG_RUN];
-#pragma unroll
-    for (int j = 0; j < LG_RUN; j++) {
-      m = fmaxf(fv[j] + m, iv[j]);
-      mv[j] = m;
+    if (lane == 31) { wF[warp] = F; wM[warp] = M; }
+    __syncthreads();
+    float before = m0;                                // what the warps before this one make of m0
+    for (int w = 0; w < warp; w++) before = fmaxf(wF[w] + before, wM[w]);
+    const float m = fmaxf(F + before, M);
+    if (tid == 0) ms[0] = m0;
+    ms[tid + 1] = m;
+    __syncthreads();
+    if (t < t1) {
+      const size_t at = (size_t)t * H + h;
+      g[at] = expf(f + (ms[tid] - m));
+      in[at] = expf(i - m);
+      low[at] = expf(-m);
     }
-    float before = __shfl_up_sync(0xffffffffu, m, 1); // as the lane before hands it on
-    if (!lane) before = m0;
-#pragma unroll
-    for (int j = 0; j < LG_RUN; j++) {
-      const int t = tb + lane * LG_RUN + j;
-      if (t < t1) {
-        const size_t at = (size_t)t * H + h;
-        g[at] = expf(fv[j] + (before - mv[j]));
-        in[at] = expf(iv[j] - mv[j]);
-        low[at] = expf(-mv[j]);
-      }
-      before = mv[j];
-    }
-    m0 = __shfl_sync(0xffffffffu, m, 31);
+    m0 = ms[LG_TOKENS];
   }
-  if (write_state && lane == 0) *kept = m0;
+  if (write_state && tid == 0) *kept = m0;
 }
 
 // From the logits' columns of u: g = e^(f + m - m'), in = e^(i - m') and low = e^-m', float32 [T, H]; the maxima of the
@@ -294,7 +286,7 @@ extern "C" int qd_linear_exp_gates(const float* u, long long ld, int i_off, int 
   if (T <= 0 || n_requests <= 0) return 0;
   if (H <= 0 || n_requests > 65535 || !ib || !fb || !(cap > 0.f) || !state || !g || !in || !low) return QD_ERR_UNSUPPORTED;
   const ExpGates a = {u, ld, i_off, f_off, ib, fb, cap, m_off, 1};
-  qd_launch(linear_exp_gates_kernel, dim3(H, n_requests), dim3(32), 0, stream, a, H, state, state_stride, cu_tokens, slots,
+  qd_launch(linear_exp_gates_kernel, dim3(H, n_requests), dim3(LG_TOKENS), 0, stream, a, H, state, state_stride, cu_tokens, slots,
             write_state, g, in, low);
   return qd_last_error();
 }
@@ -495,7 +487,14 @@ linear_scan_kernel(LinearScan a, float* __restrict__ out) {
   constexpr int THREADS = 8 * COLS / CPT, E = DP / 8, RUN = 8 / CPT;
   extern __shared__ __align__(16) float ls_sm[];      // two stages
   const int tid = threadIdx.x, x = tid & 7, jl = (tid >> 3) * CPT;
-  const int h = blockIdx.y, req = blockIdx.z, j0 = blockIdx.x * COLS, j = j0 + jl;
+  // a CTA that holds nothing but a normaliser has little to do: those come last, beside others
+  int h = blockIdx.y, piece = blockIdx.x;
+  if (a.nrm && a.dv % COLS == 0) {
+    const int b = h * gridDim.x + piece, full = gridDim.x - 1;
+    h = b < a.H * full ? b / full : b - a.H * full;
+    piece = b < a.H * full ? b - h * full : full;
+  }
+  const int req = blockIdx.z, j0 = piece * COLS, j = j0 + jl;
   const int gk = h / (a.H / a.G), d = a.d, dv = a.dv, nc = dv + a.nrm;
   const int t0 = a.cu_tokens[req], t1 = a.cu_tokens[req + 1];
   if (t0 >= t1) return;
@@ -815,7 +814,7 @@ linear_step_kernel(LinearScan a, LinearFinish f, ExpGates eg) {
   float g, in = 1.f, m = 0.f;
   if (!DELTA && eg.on) {
     float i, lf;
-    exp_gate_logs(eg, t, h, i, lf);
+    exp_gate_logs(eg, eg.u[(size_t)t * eg.ld + eg.i_off + h], eg.u[(size_t)t * eg.ld + eg.f_off + h], h, i, lf);
     const float m0 = kept[eg.m_off + h];
     m = fmaxf(lf + m0, i);
     g = expf(lf + (m0 - m));
@@ -907,14 +906,15 @@ extern "C" int qd_linear_scan(const float* q, const float* k, const float* v, lo
   // as many columns at a time as make the turns even
   const int most = LS_STEP_THREADS(DP) / 4, turns = (nc + most - 1) / most, cols = ((nc + turns - 1) / turns + 7) / 8 * 8;
   const size_t step_smem = ((size_t)nc + 40) * sizeof(float);
-  // few heads: half as many columns to a CTA, so that more multiprocessors work
+  // few heads: half as many columns to a CTA, so that more multiprocessors work (the CTA of a normaliser's single column
+  // costs next to nothing)
   static int sms = 0;
   if (!sms) {
     int dev = 0;
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   }
-  const bool narrow = (long long)((nc + 31) / 32) * H * n_requests * 2 <= sms + sms / 8;
+  const bool narrow = (long long)((dv + 31) / 32) * H * n_requests * 2 <= sms + sms / 8;
 #define LS_LAUNCH(KERNEL, COLS, THREADS, FLOATS)                                                                     \
   do {                                                                                                                \
     const size_t smem = (size_t)(FLOATS) * sizeof(float);                                                             \

@@ -772,24 +772,30 @@ def latent_attend(qcat: torch.Tensor, cache: torch.Tensor, block_table: torch.Te
 
 
 def latent_gather(cache: torch.Tensor, block_table: torch.Tensor, cu_tokens: torch.Tensor, start_pos: torch.Tensor,
-                  n_requests: int, r: int, out: torch.Tensor, Lmax: int) -> None:
-    """out[q * Lmax + j] = the first ``r`` elements of cached row j of request q, for every row of the request's context
-    (what it holds and this step's tokens); rows past it are zero.  ``cache`` [pages, page_size, W]."""
+                  n_requests: int, r: int, out: torch.Tensor, Lmax: int, window: int = 0) -> None:
+    """out[q * Lmax + j] = the first ``r`` elements of cached row lo + j of request q, for every row of the request's context
+    (what it holds and this step's tokens) from lo on: 0, or with ``window`` the first row that the portion's first token
+    sees; rows past the context are zero.  ``cache`` [pages, page_size, W]."""
     assert out.shape == (n_requests * Lmax, r) and out.dtype == cache.dtype and cache.dim() == 3
     assert block_table.dtype == torch.int32 and block_table.dim() == 2 and block_table.shape[0] >= n_requests
     _contig(cache, "cache"); _contig(block_table, "block_table"); _contig(out, "out")
     _check(library("latent_attention").qd_latent_gather(
         _ptr(cache), _I(dtype_code(cache.dtype)), _ptr(block_table), _I(block_table.shape[1]), _ptr(cu_tokens),
-        _ptr(start_pos), _I(n_requests), _I(cache.shape[1]), _I(cache.shape[2]), _I(r), _ptr(out), _I(Lmax), _stream()),
-        "latent_gather")
+        _ptr(start_pos), _I(n_requests), _I(cache.shape[1]), _I(cache.shape[2]), _I(r), _ptr(out), _I(Lmax), _I(window),
+        _stream()), "latent_gather")
 
 
-def round_rows(x: torch.Tensor, out: torch.Tensor) -> None:
-    """out = x rounded to bfloat16; x float32 [T, N] (a column range of a wider buffer is fine), out dense."""
-    assert x.dtype == torch.float32 and out.dtype == torch.bfloat16 and x.shape == out.shape and x.stride(1) == 1
+def latent_queries(q: torch.Tensor, out: torch.Tensor, H: int, dn: int, dr: int, cos: torch.Tensor, sin: torch.Tensor,
+                   rot_dims: int, positions: torch.Tensor, pairing: int = 0) -> None:
+    """out[t, h] = [unrotated part (dn) | rotated part (dr) turned by the token's position], rounded to bfloat16; q float32
+    [T, H * (dn + dr)] (a column range of a wider buffer is fine), out dense."""
+    T = q.shape[0]
+    assert q.dtype == torch.float32 and out.dtype == torch.bfloat16 and q.shape == out.shape == (T, H * (dn + dr))
+    assert q.stride(1) == 1 and cos.shape[1] == rot_dims // 2
     _contig(out, "out")
-    _check(library("latent_attention").qd_round_rows(_ptr(x), _LL(x.stride(0)), _ptr(out), _I(x.shape[0]),
-                                                     _I(x.shape[1]), _stream()), "round_rows")
+    _check(library("latent_attention").qd_latent_queries(
+        _ptr(q), _LL(q.stride(0)), _ptr(out), _I(T), _I(H), _I(dn), _I(dr), _ptr(cos), _ptr(sin), _I(rot_dims), _I(pairing),
+        _ptr(positions), _stream()), "latent_queries")
 
 
 def latent_expand(o_lat: torch.Tensor, wuv: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor,
@@ -1301,10 +1307,10 @@ SINK_MMA_ROWS = 64       # rows, (token, head within the group) pairs, of one ti
 
 
 def sink_mma_supported(dtype: torch.dtype, H: int, G: int, d: int, vd: int) -> bool:
-    """What the tensor-core form of the sink attention takes: bfloat16, head sizes that are multiples of 8 up to 128,
-    groups of up to 64 query heads per key/value head; any page size."""
+    """What the tensor-core form of the sink attention takes: bfloat16, head sizes that are multiples of 8 up to 192
+    (keys) and 128 (values), groups of up to 64 query heads per key/value head; any page size."""
     return (dtype == torch.bfloat16 and H % G == 0 and H // G <= SINK_MMA_ROWS and d % 8 == 0 and vd % 8 == 0
-            and 0 < d <= 128 and 0 < vd <= 128)
+            and 0 < d <= 192 and 0 < vd <= 128)
 
 
 def sink_attention_mma(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, block_table: torch.Tensor,

@@ -117,31 +117,42 @@ class LatentAttention(Mixer):
         self.w_uk_twice = torch.cat((uk, uk), dim=1).contiguous() if dtype == torch.bfloat16 else None
         self.w_uv_twice = torch.cat((uv, uv), dim=1).contiguous() if dtype == torch.bfloat16 else None
         self._no_table = torch.zeros((1, 0), dtype=torch.float32, device=device)
-        # the expanded form's one matrix: a row of context -> [keys of all heads | values of all heads]
-        self.w_ukv = torch.cat((self.w_uk, self.w_uv), dim=0).contiguous() if self._can_expand(dtype) else None
+        # the expanded form's one matrix: a cached row [c | kr] -> [keys of all heads, each [Wuk_h c | kr] | values of all heads]
+        self.w_ukv = None
+        if self._can_expand(dtype):
+            r, dr = self.kv_rank, self.rope_dim
+            keys = torch.zeros((H, self.nope_dim + dr, r + dr), dtype=dtype, device=device)
+            keys[:, :self.nope_dim, :r] = uk
+            keys[:, self.nope_dim:, r:] = torch.eye(dr, dtype=dtype, device=device)
+            values = torch.zeros((H * self.v_dim, r + dr), dtype=dtype, device=device)
+            values[:, :r] = self.w_uv
+            self.w_ukv = torch.cat((keys.view(-1, r + dr), values), dim=0).contiguous()
 
     def _can_expand(self, dtype) -> bool:
-        return (dtype == torch.bfloat16 and self.rope_dim == 0 and not self.output_gate and not self.window
-                and kernels.sink_mma_supported(dtype, self.num_heads, self.num_heads, self.nope_dim, self.v_dim))
+        return (dtype == torch.bfloat16 and not self.output_gate and (self.kv_rank + self.rope_dim) % 8 == 0
+                and kernels.sink_mma_supported(dtype, self.num_heads, self.num_heads, self.nope_dim + self.rope_dim, self.v_dim))
 
     def _attend_expanded(self, q: torch.Tensor, attn: torch.Tensor, ctx, cache: PagedCacheView, nd: int,
                          lmax: int) -> None:
         """Requests nd.. of the step (rows cu_tokens[nd].. of q and attn): gather their contexts' rows, expand keys
         and values, attend with the tensor-core kernel for heads that each have their own keys (a page of one key:
-        [keys of all heads | values of all heads] is a row of the product)."""
-        H, dn, dv, r = self.num_heads, self.nope_dim, self.v_dim, self.kv_rank
+        [keys of all heads | values of all heads] is a row of the product).  In a window only the rows that the portion's
+        first token still sees are expanded, and positions count from the first of them."""
+        H, dn, dr, dv = self.num_heads, self.nope_dim, self.rope_dim, self.v_dim
+        W, d, window, pos = self.kv_rank + dr, dn + dr, self.window or 0, self.position
+        rot = (pos.cos, pos.sin, pos.rotary_dim) if pos is not None else (self._no_table, self._no_table, 0)
         R = ctx.num_requests - nd
         T = q.shape[0]
-        qb = torch.empty((T, H * dn), dtype=torch.bfloat16, device=q.device)
-        kernels.round_rows(q, qb)
-        rows = torch.empty((R * lmax, r), dtype=torch.bfloat16, device=q.device)
-        kernels.latent_gather(cache.kv, cache.group.block_table[nd:], ctx.cu_tokens[nd:], ctx.start_pos[nd:], R, r,
-                              rows, lmax)
-        kv = torch.empty((R * lmax, H * (dn + dv)), dtype=torch.bfloat16, device=q.device)
+        qb = torch.empty((T, H * d), dtype=torch.bfloat16, device=q.device)
+        kernels.latent_queries(q, qb, H, dn, dr, *rot, ctx.positions, pairing=pos.pairing_code if pos is not None else 0)
+        rows = torch.empty((R * lmax, W), dtype=torch.bfloat16, device=q.device)
+        start = ctx.start_pos[nd:]
+        kernels.latent_gather(cache.kv, cache.group.block_table[nd:], ctx.cu_tokens[nd:], start, R, W, rows, lmax, window)
+        kv = torch.empty((R * lmax, H * (d + dv)), dtype=torch.bfloat16, device=q.device)
         matmul_backend.linear(rows, self.w_ukv, None, kv)
         table = torch.arange(R * lmax, dtype=torch.int32, device=q.device).view(R, lmax)
-        kernels.sink_attention_mma(qb, attn, kv, table, ctx.cu_tokens[nd:], ctx.start_pos[nd:], R,
-                                   T - int(ctx.host_cu_tokens[nd]), H, H, dn, dv, 1, self.scale, 0, None)
+        kernels.sink_attention_mma(qb, attn, kv, table, ctx.cu_tokens[nd:], start.clamp(max=window - 1) if window else start, R,
+                                   T - int(ctx.host_cu_tokens[nd]), H, H, d, dv, 1, self.scale, window, None)
 
     def forward(self, x: torch.Tensor, ctx, cache: PagedCacheView) -> torch.Tensor:
         T, H = x.shape[0], self.num_heads
@@ -159,9 +170,10 @@ class LatentAttention(Mixer):
         Ta = T
         if self.w_ukv is not None and not ctx.all_decode and ctx.max_portion >= EXPAND_TOKENS:
             nd = getattr(ctx, "num_decode", 0)
-            lmax = max(s + c1 - c0 for s, c0, c1 in zip(ctx.host_start_pos[nd:], ctx.host_cu_tokens[nd:],
+            held = lambda s: min(s, self.window - 1) if self.window else s      # cached rows that the portion still sees
+            lmax = max(held(s) + c1 - c0 for s, c0, c1 in zip(ctx.host_start_pos[nd:], ctx.host_cu_tokens[nd:],
                                                               ctx.host_cu_tokens[nd + 1:]))
-            if (ctx.num_requests - nd) * lmax * H * (dn + dv) * 2 <= EXPAND_MAX_BYTES:
+            if (ctx.num_requests - nd) * lmax * H * (dn + dr + dv) * 2 <= EXPAND_MAX_BYTES:
                 self._attend_expanded(q, attn, ctx, cache, nd, lmax)
                 Ta = nd
         if Ta:
