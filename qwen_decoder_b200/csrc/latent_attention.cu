@@ -21,12 +21,15 @@
 template <typename T> struct Vec16;
 template <> struct Vec16<float> {
   static constexpr int N = 4;
+  __device__ static void unpack(const uint4& v, float* o) {
+    o[0] = __uint_as_float(v.x); o[1] = __uint_as_float(v.y); o[2] = __uint_as_float(v.z); o[3] = __uint_as_float(v.w);
+  }
   __device__ static void load(const float* p, float* o) { float4 v = *reinterpret_cast<const float4*>(p); o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w; }
 };
 template <> struct Vec16<bf16> {
   static constexpr int N = 8;
-  __device__ static void load(const bf16* p, float* o) {
-    uint4 v = *reinterpret_cast<const uint4*>(p);
+  __device__ static void load(const bf16* p, float* o) { unpack(*reinterpret_cast<const uint4*>(p), o); }
+  __device__ static void unpack(const uint4& v, float* o) {
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
 #pragma unroll
     for (int i = 0; i < 4; i++) { o[2 * i] = __low2float(h[i]); o[2 * i + 1] = __high2float(h[i]); }
@@ -48,6 +51,7 @@ __device__ __forceinline__ float la_turn(const float* x, int e, int half, int pa
 #define LA_TILE 32          // keys per staged tile
 #define LA_MAX_R 512        // latent size the attend kernel takes (16 accumulators a lane)
 #define LA_TT 8             // tokens per CTA in absorb and expand
+#define LA_AHEAD 8          // rows of weights a thread of the vectorised absorb asks for ahead of time
 
 // ----------------------------------------------------------------------------- prep
 // u row t (float32, stride ldu): columns [q_off, q_off + q_rank) the raw query latent (q_rank 0: the design has
@@ -133,8 +137,9 @@ latent_absorb_kernel(const float* __restrict__ q, long long ldq, const TW* __res
 }
 
 // The same with 16-byte loads of Wuk, for latent sizes whose pieces divide the CTA evenly (a share's r / V a divisor of 256):
-// thread (jg, dg) owns V consecutive latent columns and every (256 * V / r)-th unrotated dimension; the groups'
-// partial sums meet in shared memory.  grid (token tiles, heads, shares of the r columns).
+// thread (jg, dg) owns V consecutive latent columns and every DG-th unrotated dimension, DG the number of groups; the
+// first LA_AHEAD rows of its weights are asked for before the kernel waits for its predecessor (no kernel of a step writes
+// them).  The groups' partial sums meet in shared memory, four tokens at a time.  grid (token tiles, heads, shares of the r columns).
 template <typename TW>
 __global__ void __launch_bounds__(256)
 latent_absorb_vec_kernel(const float* __restrict__ q, long long ldq, const TW* __restrict__ wuk,
@@ -142,52 +147,64 @@ latent_absorb_vec_kernel(const float* __restrict__ q, long long ldq, const TW* _
                          const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims,
                          const int* __restrict__ positions, int pairing) {
   pdl_launch_dependents();
-  pdl_wait();
   constexpr int V = Vec16<TW>::N;
-  extern __shared__ float sm[];
-  float* qs = sm;                              // [LA_TT][dn]
-  float* red = sm + LA_TT * dn;                // [LA_TT][rs]
+  extern __shared__ __align__(16) float sm[];
+  float* red = sm;                             // [DG][4][rs] = 1024 V floats
+  float* qs = sm + 1024 * V;                   // [LA_TT][dn]
   const int h = blockIdx.y, t0 = blockIdx.x * LA_TT;
   const int nt = min(LA_TT, T - t0);
   const int W = r + dr, rs = r / gridDim.z, j0 = blockIdx.z * rs;      // this CTA's columns
+  const int JG = rs / V, DG = 256 / JG;
+  const int jg = threadIdx.x % JG, dg = threadIdx.x / JG;
+  const TW* wbase = wuk + (size_t)h * dn * r + j0 + jg * V;
+  uint4 ahead[LA_AHEAD];
+#pragma unroll
+  for (int k = 0; k < LA_AHEAD; k++)
+    ahead[k] = dg + DG * k < dn ? *reinterpret_cast<const uint4*>(wbase + (size_t)(dg + DG * k) * r) : make_uint4(0, 0, 0, 0);
+  pdl_wait();
   const size_t qw = (size_t)ldq;              // q's rows are ldq floats apart (a column range of a wider buffer is fine)
   for (int i = threadIdx.x; i < LA_TT * dn; i += blockDim.x) {
     int tt = i / dn, d = i - tt * dn;
     qs[i] = tt < nt ? q[(size_t)(t0 + tt) * qw + (size_t)h * (dn + dr) + d] : 0.f;
   }
-  for (int i = threadIdx.x; i < LA_TT * rs; i += blockDim.x) red[i] = 0.f;
   __syncthreads();
-  const int JG = rs / V, DG = 256 / JG;
-  const int jg = threadIdx.x % JG, dg = threadIdx.x / JG;
   float acc[LA_TT][V];
 #pragma unroll
   for (int tt = 0; tt < LA_TT; tt++)
 #pragma unroll
     for (int v = 0; v < V; v++) acc[tt][v] = 0.f;
-  const TW* wbase = wuk + (size_t)h * dn * r + j0 + jg * V;
-#pragma unroll 4
-  for (int d = dg; d < dn; d += DG) {
+  auto add = [&](const uint4& raw, int d) {
     float w[V];
-    Vec16<TW>::load(wbase + (size_t)d * r, w);
+    Vec16<TW>::unpack(raw, w);
 #pragma unroll
     for (int tt = 0; tt < LA_TT; tt++) {
       const float qv = qs[tt * dn + d];
 #pragma unroll
       for (int v = 0; v < V; v++) acc[tt][v] = fmaf(qv, w[v], acc[tt][v]);
     }
-  }
-  for (int turn = 0; turn < DG; turn++) {        // the groups add in turn: the order of additions is fixed
-    if (dg == turn) {
+  };
 #pragma unroll
-      for (int tt = 0; tt < LA_TT; tt++)
+  for (int k = 0; k < LA_AHEAD; k++)
+    if (dg + DG * k < dn) add(ahead[k], dg + DG * k);
+#pragma unroll 4
+  for (int d = dg + DG * LA_AHEAD; d < dn; d += DG) add(*reinterpret_cast<const uint4*>(wbase + (size_t)d * r), d);
 #pragma unroll
-        for (int v = 0; v < V; v++) red[tt * rs + jg * V + v] += acc[tt][v];
+  for (int part = 0; part < LA_TT / 4; part++) {  // the groups are added in order
+    if (part * 4 >= nt) break;                   // the same for the whole CTA
+#pragma unroll
+    for (int tt = 0; tt < 4; tt++)
+#pragma unroll
+      for (int v = 0; v < V; v += 4)
+        *reinterpret_cast<float4*>(red + ((size_t)dg * 4 + tt) * rs + jg * V + v) =
+            make_float4(acc[part * 4 + tt][v], acc[part * 4 + tt][v + 1], acc[part * 4 + tt][v + 2], acc[part * 4 + tt][v + 3]);
+    __syncthreads();
+    for (int i = threadIdx.x; i < 4 * rs; i += blockDim.x) {
+      const int tt = i / rs, j = i - tt * rs;
+      float sum = 0.f;
+      for (int g = 0; g < DG; g++) sum += red[((size_t)g * 4 + tt) * rs + j];
+      if (part * 4 + tt < nt) qcat[((size_t)(t0 + part * 4 + tt) * H + h) * W + j0 + j] = sum;
     }
     __syncthreads();
-  }
-  for (int i = threadIdx.x; i < nt * rs; i += blockDim.x) {
-    int tt = i / rs, j = i - tt * rs;
-    qcat[((size_t)(t0 + tt) * H + h) * W + j0 + j] = red[i];
   }
   if (blockIdx.z != 0) return;
   const int half = rot_dims >> 1;
@@ -598,6 +615,75 @@ latent_expand_kernel(const float* __restrict__ o_lat, const TW* __restrict__ wuv
   }
 }
 
+// The same for rows in 16-byte pieces of up to 512 elements (NP pieces a lane): the four rows of Wuv a warp takes are asked for
+// before the kernel waits for its predecessor, and a row's sums over eight tokens are added up by one exchange.
+template <typename TW, typename TO, int NP>
+__global__ void __launch_bounds__(256)
+latent_expand_vec_kernel(const float* __restrict__ o_lat, const TW* __restrict__ wuv, const float* __restrict__ gate,
+                         long long ldg, TO* __restrict__ out, int T, int H, int dv, int r) {
+  pdl_launch_dependents();
+  constexpr int V = Vec16<TW>::N;
+  extern __shared__ __align__(16) float os[];  // [LA_TT][r]
+  const int h = blockIdx.y, t0 = blockIdx.x * LA_TT, nt = min(LA_TT, T - t0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  uint4 raw[4][NP];
+#pragma unroll
+  for (int k = 0; k < 4; k++)
+#pragma unroll
+    for (int p = 0; p < NP; p++) {
+      const int i = blockIdx.z * 32 + warp + 8 * k, j = (p * 32 + lane) * V;
+      raw[k][p] = i < dv && j < r ? *reinterpret_cast<const uint4*>(wuv + ((size_t)h * dv + i) * r + j) : make_uint4(0, 0, 0, 0);
+    }
+  pdl_wait();
+  const int r4 = r >> 2;
+  for (int i = threadIdx.x; i < LA_TT * r4; i += 256) {
+    const int tt = i / r4, j = (i - tt * r4) * 4;
+    *reinterpret_cast<float4*>(os + tt * r + j) =
+        tt < nt ? *reinterpret_cast<const float4*>(o_lat + ((size_t)(t0 + tt) * H + h) * r + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < 4; k++) {
+    const int i = blockIdx.z * 32 + warp + 8 * k;
+    if (i >= dv) break;                           // the same for the whole warp
+    float acc[LA_TT];
+#pragma unroll
+    for (int tt = 0; tt < LA_TT; tt++) acc[tt] = 0.f;
+#pragma unroll
+    for (int p = 0; p < NP; p++) {
+      const int j = (p * 32 + lane) * V;
+      if (j >= r) break;
+      float w[V];
+      Vec16<TW>::unpack(raw[k][p], w);
+#pragma unroll
+      for (int tt = 0; tt < LA_TT; tt++)
+#pragma unroll
+        for (int v = 0; v < V; v += 4) {
+          const float4 o = *reinterpret_cast<const float4*>(os + tt * r + j + v);
+          acc[tt] = fmaf(w[v], o.x, fmaf(w[v + 1], o.y, fmaf(w[v + 2], o.z, fmaf(w[v + 3], o.w, acc[tt]))));
+        }
+    }
+    // after the step with distance o a lane keeps the sums of the half of the tokens that its bit o names
+#pragma unroll
+    for (int o = 16, n = LA_TT / 2; n > 0; o >>= 1, n >>= 1) {
+      const bool upper = lane & o;
+#pragma unroll
+      for (int c = 0; c < n; c++) {
+        const float send = upper ? acc[c] : acc[c + n], keep = upper ? acc[c + n] : acc[c];
+        acc[c] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+      }
+    }
+    acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 2);
+    acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
+    const int tt = (lane & 16 ? 4 : 0) + (lane & 8 ? 2 : 0) + (lane & 4 ? 1 : 0);
+    if ((lane & 3) == 0 && tt < nt) {
+      float v = acc[0];
+      if (gate) v *= 1.0f / (1.0f + expf(-gate[(size_t)(t0 + tt) * ldg + (size_t)h * dv + i]));
+      out[(size_t)(t0 + tt) * H * dv + (size_t)h * dv + i] = from_float<TO>(v);
+    }
+  }
+}
+
 // ----------------------------------------------------------------------------- launchers
 // QD_LATENT_MMA=0 in the environment keeps the float32-FMA attend kernel in bfloat16 too (to compare the two).
 static inline bool lm_enabled() {
@@ -636,7 +722,7 @@ extern "C" int qd_latent_absorb(const float* q, long long ldq, const void* wuk, 
   if (smem > 48 * 1024 || H > 65535) return QD_ERR_UNSUPPORTED;
   {
     const int V = w_dtype == QD_F32 ? 4 : 8;
-    const size_t vsm = (size_t)LA_TT * (dn + r) * sizeof(float);
+    const size_t vsm = ((size_t)LA_TT * dn + 1024 * V) * sizeof(float);
     if (!pre && (w_dtype == QD_F32 || w_dtype == QD_BF16) && r % V == 0 && r / V <= 256 && 256 % (r / V) == 0 &&
         !((uintptr_t)wuk & 15) && vsm <= 48 * 1024) {
       // few tokens: a head's columns are shared among CTAs while the grid leaves multiprocessors idle
@@ -720,6 +806,16 @@ extern "C" int qd_latent_expand(const float* o_lat, const void* wuv, int w_dtype
   if (smem > 48 * 1024 || H > 65535) return QD_ERR_UNSUPPORTED;
   dim3 grid((T + LA_TT - 1) / LA_TT, H, (dv + 31) / 32);
   const int vec = (r % (w_dtype == QD_F32 ? 4 : 8) == 0 && !((uintptr_t)wuv & 15)) ? 1 : 0;     // rows in 16-byte pieces
+  if (vec && !pre && r <= 512 && !((uintptr_t)o_lat & 15) && w_dtype == out_dtype && (w_dtype == QD_F32 || w_dtype == QD_BF16)) {
+#define LE_GO(T_, NP_)                                                                                                    \
+  qd_launch(latent_expand_vec_kernel<T_, T_, NP_>, grid, dim3(256), smem, stream, o_lat, (const T_*)wuv, gate, ldg, (T_*)out, T, \
+            H, dv, r)
+    const int np = (r + 32 * (w_dtype == QD_F32 ? 4 : 8) - 1) / (32 * (w_dtype == QD_F32 ? 4 : 8));
+    if (w_dtype == QD_F32) { if (np == 1) LE_GO(float, 1); else if (np == 2) LE_GO(float, 2); else LE_GO(float, 4); }
+    else { if (np == 1) LE_GO(bf16, 1); else LE_GO(bf16, 2); }
+#undef LE_GO
+    return qd_last_error();
+  }
   if (w_dtype == QD_F32 && out_dtype == QD_F32)
     qd_launch(latent_expand_kernel<float, float>, grid, dim3(256), smem, stream, o_lat, (const float*)wuv, gate, ldg,
               (float*)out, T, H, dv, r, vec, pre);

@@ -224,16 +224,16 @@ __device__ __forceinline__ void exp_gate_logs(const ExpGates& a, float ui, float
 }
 
 // grid (H, requests): the maxima of a portion by a scan over (sum of f, maximum): what a run of tokens does to m is
-// m -> max(F + m, M), and runs compose.  A thread takes one token of LG_TOKENS; warps scan their 32, then one another's.
+// m -> max(F + m, M), and runs compose.  A thread takes one token of as many as the CTA has threads; warps scan their 32, then one another's.
 // Every factor is made from the maxima as they are handed on, so what rounds in the scan cancels between a token and the next.
-#define LG_TOKENS 256
+#define LG_TOKENS 1024
 __global__ void __launch_bounds__(LG_TOKENS)
 linear_exp_gates_kernel(ExpGates a, int H, float* __restrict__ state, long long state_stride,
                         const int* __restrict__ cu_tokens, const int* __restrict__ slots, int write_state,
                         float* __restrict__ g, float* __restrict__ in, float* __restrict__ low) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float wF[LG_TOKENS / 32], wM[LG_TOKENS / 32], ms[LG_TOKENS + 1];
+  __shared__ float wF[32], wM[32], ms[LG_TOKENS + 1];
   const int h = blockIdx.x, req = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int t0 = cu_tokens[req], t1 = cu_tokens[req + 1];
   if (t0 >= t1) return;
@@ -244,11 +244,12 @@ linear_exp_gates_kernel(ExpGates a, int H, float* __restrict__ state, long long 
     if (t < t1) { ui = a.u[(size_t)t * a.ld + a.i_off + h]; uf = a.u[(size_t)t * a.ld + a.f_off + h]; }
   };
   fetch(t0 + tid);
-  for (int tb = t0; tb < t1; tb += LG_TOKENS) {
+  const int at_once = blockDim.x, warps = at_once >> 5;
+  for (int tb = t0; tb < t1; tb += at_once) {
     const int t = tb + tid;
     float i = -INFINITY, f = 0.f;                     // past the end: m stays as it is
     if (t < t1) exp_gate_logs(a, ui, uf, h, i, f);
-    fetch(t + LG_TOKENS);
+    fetch(t + at_once);
     float F = f, M = i;                               // of the warp's tokens up to this one
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -260,8 +261,15 @@ linear_exp_gates_kernel(ExpGates a, int H, float* __restrict__ state, long long 
     }
     if (lane == 31) { wF[warp] = F; wM[warp] = M; }
     __syncthreads();
-    float before = m0;                                // what the warps before this one make of m0
-    for (int w = 0; w < warp; w++) before = fmaxf(wF[w] + before, wM[w]);
+    // what the warps before this one make of m0: lane w holds warp w's run; neighbours compose, five times
+    float Fw = lane < warp && lane < warps ? wF[lane] : 0.f, Mw = lane < warp && lane < warps ? wM[lane] : -INFINITY;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float Fr = __shfl_down_sync(0xffffffffu, Fw, o), Mr = __shfl_down_sync(0xffffffffu, Mw, o);
+      Mw = fmaxf(Mw + Fr, Mr);
+      Fw += Fr;
+    }
+    const float before = fmaxf(__shfl_sync(0xffffffffu, Fw, 0) + m0, __shfl_sync(0xffffffffu, Mw, 0));
     const float m = fmaxf(F + before, M);
     if (tid == 0) ms[0] = m0;
     ms[tid + 1] = m;
@@ -272,7 +280,7 @@ linear_exp_gates_kernel(ExpGates a, int H, float* __restrict__ state, long long 
       in[at] = expf(i - m);
       low[at] = expf(-m);
     }
-    m0 = ms[LG_TOKENS];
+    m0 = ms[at_once];
   }
   if (write_state && tid == 0) *kept = m0;
 }
@@ -286,7 +294,7 @@ extern "C" int qd_linear_exp_gates(const float* u, long long ld, int i_off, int 
   if (T <= 0 || n_requests <= 0) return 0;
   if (H <= 0 || n_requests > 65535 || !ib || !fb || !(cap > 0.f) || !state || !g || !in || !low) return QD_ERR_UNSUPPORTED;
   const ExpGates a = {u, ld, i_off, f_off, ib, fb, cap, m_off, 1};
-  qd_launch(linear_exp_gates_kernel, dim3(H, n_requests), dim3(LG_TOKENS), 0, stream, a, H, state, state_stride, cu_tokens, slots,
+  qd_launch(linear_exp_gates_kernel, dim3(H, n_requests), dim3(T < LG_TOKENS ? (T + 31) / 32 * 32 : LG_TOKENS), 0, stream, a, H, state, state_stride, cu_tokens, slots,
             write_state, g, in, low);
   return qd_last_error();
 }
