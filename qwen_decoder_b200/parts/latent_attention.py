@@ -16,7 +16,8 @@ dtypes.  The plain norms here multiply by the stored weight (no offset); their e
 
 Variants, all constructor parameters: ``q_rank`` = 0 leaves the query latent out, q = Wq h (tensor ``<prefix>q``);
 ``rope_dim`` = 0 leaves the rotated part out (no position enters the scores, the cached row is c alone);
-``output_gate`` = False leaves the sigmoid gate out.
+``output_gate`` = False leaves the sigmoid gate out; ``window``: a query sees the last so many keys; the rotated parts turn
+in whichever pairs the ``position`` part says.
 """
 from __future__ import annotations
 
